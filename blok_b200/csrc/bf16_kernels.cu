@@ -366,6 +366,64 @@ int launch_bf16_gemv_splitk_pair(const uint16_t *w1, int rows1, uint16_t *y1, co
   return launch_status("bf16_gemv16_splitk_kernel<pair>");
 }
 
+// ---------------------------------------------------------------------------
+// Per-head mat-vec for up to 8 tokens: y[tok, head, r] = sum_c W[head][r][c] * x[tok, head, c].
+// grid = (rows/16, heads), 4 warps split K.  Strides are in elements.
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(128)
+    bf16_head_gemv_kernel(const uint16_t *__restrict__ w, long w_head_stride, const uint16_t *__restrict__ x,
+                          long x_tok_stride, long x_head_stride, uint16_t *__restrict__ y, long y_tok_stride,
+                          long y_head_stride, int cols, int T_all) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  __shared__ float partial[4][16][8];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int g = lane >> 2, t = lane & 3;
+  const int head = blockIdx.y;
+  // blockIdx.z: the group of 8 tokens (the later groups find the head's matrix in L2)
+  const int T = min(8, T_all - 8 * (int)blockIdx.z);
+  x += (size_t)blockIdx.z * 8 * x_tok_stride;
+  y += (size_t)blockIdx.z * 8 * y_tok_stride;
+  const int per_row = cols / 8;
+  for (int u = tid; u < per_row * T; u += blockDim.x) {
+    int tok = u / per_row, c = u - tok * per_row;
+    uint4 v = reinterpret_cast<const uint4 *>(x + (size_t)tok * x_tok_stride + (size_t)head * x_head_stride)[c];
+    reinterpret_cast<uint4 *>(smem + tok * bf16_x_row_bytes(cols))[c] = v;
+  }
+  __syncthreads();
+  const size_t wrow = cols / 8;
+  const int row0 = blockIdx.x * 16;
+  const uint4 *w_lo = reinterpret_cast<const uint4 *>(w + (size_t)head * w_head_stride) + (size_t)(row0 + g) * wrow;
+  const uint4 *w_hi = w_lo + 8 * wrow;
+  const int tok = g < T ? g : T - 1;
+  const uint4 *xrow = reinterpret_cast<const uint4 *>(smem + tok * bf16_x_row_bytes(cols)) + t;
+  const int ksteps = cols / 32;
+  const int base = ksteps / 4, rem = ksteps % 4;
+  const int ks0 = warp * base + (warp < rem ? warp : rem);
+  const int nsteps = base + (warp < rem ? 1 : 0);
+  float d[4] = {0.f, 0.f, 0.f, 0.f};
+  bf16_rows16_accumulate(w_lo, w_hi, xrow, ks0, nsteps, t, d);
+  partial[warp][g][2 * t] = d[0];
+  partial[warp][g][2 * t + 1] = d[1];
+  partial[warp][g + 8][2 * t] = d[2];
+  partial[warp][g + 8][2 * t + 1] = d[3];
+  __syncthreads();
+  if (tid < 128) {
+    int r = tid >> 3, tk = tid & 7;
+    if (tk < T) {
+      float v = partial[0][r][tk] + partial[1][r][tk] + partial[2][r][tk] + partial[3][r][tk];
+      y[(size_t)tk * y_tok_stride + (size_t)head * y_head_stride + row0 + r] = f32_to_bf16_bits(v);
+    }
+  }
+}
+
+int launch_head_gemv(const uint16_t *w, long w_head_stride, const uint16_t *x, long x_tok_stride,
+                            long x_head_stride, uint16_t *y, long y_tok_stride, long y_head_stride, int rows, int cols,
+                            int heads, int T, cudaStream_t stream) {
+  size_t smem = bf16_x_row_bytes(cols) * std::min(T, 8);
+  bf16_head_gemv_kernel<<<dim3(rows / 16, heads, (T + 7) / 8), 128, smem, stream>>>(w, w_head_stride, x, x_tok_stride, x_head_stride,
+                                                                      y, y_tok_stride, y_head_stride, cols, T);
+  return launch_status("bf16_head_gemv_kernel");
+}
 
 // mid[T, ffn] = SwiGLU front half.
 int launch_bf16_gateup(const uint16_t *gate, const uint16_t *up, const uint16_t *x, uint16_t *mid, int ffn, int cols,

@@ -1,0 +1,443 @@
+// Linear attention with a fixed decay per head and no softmax (retention, lightning attention):
+//   S_t = decay S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t                     (S fp32 [dim, vdim], per head and sequence)
+//
+// Decode runs the recurrence itself, every thread holding a few elements of S in registers.  A prompt runs in chunks of 64
+// tokens: with w_ij = decay^(i-j) for j <= i inside a chunk and S the state in front of it,
+//   o_i = sum_j w_ij (q_i . k_j) v_j + decay^(i+1) S^T q_i
+//   S'  = decay^L S + sum_j decay^(L-1-j) k_j v_j^T                        (L tokens in the chunk)
+// in three launches: every chunk's own contribution to the state in parallel, a scan over the chunks that turns the
+// contributions into the states in front of them, every chunk's output in parallel.  The products run on bf16 tensor cores
+// with their fp32 factors (scores, decays, states) split into three bf16 parts (bf16_split.cuh).
+#include "bf16_split.cuh"
+#include "stack_kernels.h"
+
+namespace blok {
+
+template <typename Act>
+__device__ __forceinline__ float la_load(const Act *p) {
+  if constexpr (sizeof(Act) == 2) return bf16_bits_to_f32(*p);
+  else return *p;
+}
+__device__ __forceinline__ float la_silu(float z) { return z / (1.0f + expf(-z)); }
+// A projection after its activation, rounded as the activation's type is.
+template <typename Act>
+__device__ __forceinline__ float la_proj(const Act *p, bool silu) {
+  const float v = la_load(p);
+  if (!silu) return v;
+  return sizeof(Act) == 2 ? round_bf16(la_silu(v)) : la_silu(v);
+}
+
+struct LaArgs {
+  const void *qkvg;
+  const float *decay_pow;
+  float *state, *o, *chunk_state;
+  const int *slot_of, *pos;  // step form
+  int slot;                  // chunk form
+  int fresh;                 // chunk form: the sequence starts here
+  int heads, dim, vdim, ld, silu, T, chunks;
+  float k_scale;
+};
+
+// ---- the recurrence: T tokens of each of gridDim.z sequences, one after the other.  CTA = 32 columns of a head's state,
+// thread = 4 columns x every 32nd row. ----
+template <typename Act, int R>
+__global__ void __launch_bounds__(256) linear_recurrent_kernel(const LaArgs a) {
+  __shared__ float sq[32 * R], sk[32 * R];
+  __shared__ float4 s_red[8][8];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, c4 = tid & 7, rg = tid >> 3;
+  const int h = blockIdx.y, b = blockIdx.z, col = blockIdx.x * 32 + c4 * 4;
+  const bool in_col = col < a.vdim;
+  const int slot = a.slot_of ? a.slot_of[b] : a.slot;
+  const bool fresh = a.slot_of ? a.pos[b] == 0 : a.fresh != 0;
+  const float decay = a.decay_pow[h * (kLinChunk + 1) + 1];
+  const int hd = a.heads * a.dim;
+  float *st = a.state + ((size_t)slot * a.heads + h) * a.dim * a.vdim + col;
+  float4 s[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = rg + 32 * r;
+    s[r] = !fresh && in_col && i < a.dim ? *reinterpret_cast<const float4 *>(st + (size_t)i * a.vdim) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  for (int t = 0; t < a.T; ++t) {
+    const size_t row = (size_t)b * a.T + t;
+    const Act *p = static_cast<const Act *>(a.qkvg) + row * a.ld + (size_t)h * a.dim;
+    if (tid < 32 * R) {
+      const bool in = tid < a.dim;
+      sq[tid] = in ? la_proj(p + tid, a.silu) : 0.f;
+      sk[tid] = in ? la_proj(p + hd + tid, a.silu) * a.k_scale : 0.f;
+    }
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (in_col) {
+      const Act *pv = static_cast<const Act *>(a.qkvg) + row * a.ld + 2 * (size_t)hd + (size_t)h * a.vdim + col;
+      v = make_float4(la_proj(pv, a.silu), la_proj(pv + 1, a.silu), la_proj(pv + 2, a.silu), la_proj(pv + 3, a.silu));
+    }
+    __syncthreads();
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const float k = sk[rg + 32 * r], q = sq[rg + 32 * r];
+      s[r] = make_float4(fmaf(decay, s[r].x, k * v.x), fmaf(decay, s[r].y, k * v.y), fmaf(decay, s[r].z, k * v.z), fmaf(decay, s[r].w, k * v.w));
+      o = make_float4(fmaf(q, s[r].x, o.x), fmaf(q, s[r].y, o.y), fmaf(q, s[r].z, o.z), fmaf(q, s[r].w, o.w));
+    }
+#pragma unroll
+    for (int d = 8; d < 32; d <<= 1) {
+      o.x += __shfl_xor_sync(0xffffffffu, o.x, d);
+      o.y += __shfl_xor_sync(0xffffffffu, o.y, d);
+      o.z += __shfl_xor_sync(0xffffffffu, o.z, d);
+      o.w += __shfl_xor_sync(0xffffffffu, o.w, d);
+    }
+    if (lane < 8) s_red[warp][lane] = o;
+    __syncthreads();
+    if (tid < 8 && in_col) {
+      float4 u = s_red[0][tid];
+#pragma unroll
+      for (int w = 1; w < 8; ++w) u = make_float4(u.x + s_red[w][tid].x, u.y + s_red[w][tid].y, u.z + s_red[w][tid].z, u.w + s_red[w][tid].w);
+      *reinterpret_cast<float4 *>(a.o + row * a.heads * a.vdim + (size_t)h * a.vdim + col) = u;
+    }
+  }
+  if (in_col) {
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (rg + 32 * r < a.dim) *reinterpret_cast<float4 *>(st + (size_t)(rg + 32 * r) * a.vdim) = s[r];
+  }
+}
+
+// ---- chunked form ----
+constexpr int kLcThreads = 128;
+constexpr int kLcCols = 64;  // columns of v per CTA
+constexpr int kLcVPitch = kLcCols * 2 + 16;
+
+// `n` rows of `cols` bf16 (a multiple of 8) from p (row pitch ld elements) into a tile; rows past n are zero.
+__device__ __forceinline__ void lc_stage(unsigned char *dst, int pitch, const uint16_t *p, int ld, int n, int cols, bool silu) {
+  const int per = cols / 8;
+  for (int u = threadIdx.x; u < kLinChunk * per; u += kLcThreads) {
+    const int r = u / per, c = u - r * per;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (r < n) {
+      v = *reinterpret_cast<const uint4 *>(p + (size_t)r * ld + c * 8);
+      if (silu) {
+        uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[j] = pack_bf16x2(la_silu(bf16lo(w[j])), la_silu(bf16hi(w[j])));
+        v = make_uint4(w[0], w[1], w[2], w[3]);
+      }
+    }
+    *reinterpret_cast<uint4 *>(dst + (size_t)r * pitch + c * 16) = v;
+  }
+}
+
+// chunk_state[c][h] = sum_j k_scale decay^(L-1-j) k_j v_j^T.  grid = (chunks, heads, columns / 64)
+__global__ void __launch_bounds__(kLcThreads) linear_chunk_state_kernel(const LaArgs a) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  const int c = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * kLcCols;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int n = min(kLinChunk, a.T - c * kLinChunk), vc = min(kLcCols, a.vdim - v0);
+  const int kp = a.dim * 2 + 16;  // pitch of the key tiles
+  unsigned char *Vs = smem + (size_t)kSplitParts * kLinChunk * kp;
+  const float *pw = a.decay_pow + h * (kLinChunk + 1);
+  const uint16_t *rows = static_cast<const uint16_t *>(a.qkvg) + (size_t)c * kLinChunk * a.ld;
+  const uint16_t *k = rows + (size_t)a.heads * a.dim + (size_t)h * a.dim;
+  for (int u = threadIdx.x; u < kLinChunk * (a.dim / 8); u += kLcThreads) {  // the decayed keys in three parts
+    const int r = u / (a.dim / 8), col = (u - r * (a.dim / 8)) * 8;
+    uint32_t part[4][kSplitParts] = {};
+    if (r < n) {
+      const uint4 x = *reinterpret_cast<const uint4 *>(k + (size_t)r * a.ld + col);
+      const uint32_t w[4] = {x.x, x.y, x.z, x.w};
+      const float wt = a.k_scale * pw[n - 1 - r];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float lo = bf16lo(w[j]), hi = bf16hi(w[j]);
+        if (a.silu) lo = round_bf16(la_silu(lo)), hi = round_bf16(la_silu(hi));
+        split_pair(lo * wt, hi * wt, part[j]);
+      }
+    }
+#pragma unroll
+    for (int p = 0; p < kSplitParts; ++p)
+      *reinterpret_cast<uint4 *>(smem + (size_t)(p * kLinChunk + r) * kp + col * 2) = make_uint4(part[0][p], part[1][p], part[2][p], part[3][p]);
+  }
+  lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)a.heads * a.dim + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
+  __syncthreads();
+  const uint32_t ks = (uint32_t)__cvta_generic_to_shared(smem), vs = (uint32_t)__cvta_generic_to_shared(Vs);
+  float *out = a.chunk_state + (((size_t)c * a.heads + h) * a.dim) * a.vdim + v0;
+  const int g = lane >> 2, t = lane & 3;
+  for (int m0 = warp * 16; m0 < a.dim; m0 += 64) {
+    float acc[kLcCols / 8][4] = {};
+#pragma unroll
+    for (int k0 = 0; k0 < kLinChunk; k0 += 16) {
+      uint32_t fa[kSplitParts][4];
+#pragma unroll
+      for (int p = 0; p < kSplitParts; ++p) ldsm4_t(frag_a_t(ks + p * kLinChunk * kp, m0, k0, kp, lane), fa[p][0], fa[p][1], fa[p][2], fa[p][3]);
+#pragma unroll
+      for (int nt = 0; nt < kLcCols / 8; nt += 2) {
+        if (nt * 8 < vc) {
+          uint32_t b0, b1, b2, b3;
+          ldsm4_t(frag_b_t(vs, nt * 8, k0, kLcVPitch, lane), b0, b1, b2, b3);
+#pragma unroll
+          for (int p = 0; p < kSplitParts; ++p) {
+            mma_bf16_16816(acc[nt], fa[p][0], fa[p][1], fa[p][2], fa[p][3], b0, b1);
+            mma_bf16_16816(acc[nt + 1], fa[p][0], fa[p][1], fa[p][2], fa[p][3], b2, b3);
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int nt = 0; nt < kLcCols / 8; ++nt) {
+      const int col = nt * 8 + 2 * t;
+      if (nt * 8 < vc) {
+        *reinterpret_cast<float2 *>(out + (size_t)(m0 + g) * a.vdim + col) = make_float2(acc[nt][0], acc[nt][1]);
+        *reinterpret_cast<float2 *>(out + (size_t)(m0 + g + 8) * a.vdim + col) = make_float2(acc[nt][2], acc[nt][3]);
+      }
+    }
+  }
+}
+
+// chunk_state[c] <- the state in front of chunk c; state <- the state behind the last chunk.
+__global__ void __launch_bounds__(128) linear_scan_kernel(const LaArgs a) {
+  const int h = blockIdx.y, i = (blockIdx.x * blockDim.x + threadIdx.x) * 4, n = a.dim * a.vdim;
+  if (i >= n) return;
+  const float *pw = a.decay_pow + h * (kLinChunk + 1);
+  float4 *st = reinterpret_cast<float4 *>(a.state + ((size_t)a.slot * a.heads + h) * n + i);
+  float4 s = a.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *st;
+  constexpr int kAhead = 4;  // chunks' loads in flight
+  const size_t stride = (size_t)a.heads * n / 4;
+  float4 *p = reinterpret_cast<float4 *>(a.chunk_state + (size_t)h * n + i);
+  for (int c0 = 0; c0 < a.chunks; c0 += kAhead) {
+    float4 own[kAhead];
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j)
+      if (c0 + j < a.chunks) own[j] = p[(size_t)(c0 + j) * stride];
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j)
+      if (c0 + j < a.chunks) {
+        const float d = pw[min(kLinChunk, a.T - (c0 + j) * kLinChunk)];
+        p[(size_t)(c0 + j) * stride] = s;
+        s = make_float4(fmaf(d, s.x, own[j].x), fmaf(d, s.y, own[j].y), fmaf(d, s.z, own[j].z), fmaf(d, s.w, own[j].w));
+      }
+  }
+  *st = s;
+}
+
+// grid = (chunks, heads, columns / 64); a warp owns 16 tokens of the chunk.
+__global__ void __launch_bounds__(kLcThreads) linear_chunk_out_kernel(const LaArgs a) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  __shared__ float s_pw[kLinChunk + 1];
+  const int c = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * kLcCols;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+  const int n = min(kLinChunk, a.T - c * kLinChunk), vc = min(kLcCols, a.vdim - v0);
+  const int kp = a.dim * 2 + 16;
+  unsigned char *Ks = smem + (size_t)kLinChunk * kp, *Vs = Ks + (size_t)kLinChunk * kp, *Ss = Vs + (size_t)kLinChunk * kLcVPitch;
+  const uint16_t *rows = static_cast<const uint16_t *>(a.qkvg) + (size_t)c * kLinChunk * a.ld;
+  const int hd = a.heads * a.dim;
+  if (threadIdx.x <= kLinChunk) s_pw[threadIdx.x] = a.decay_pow[h * (kLinChunk + 1) + threadIdx.x];
+  lc_stage(smem, kp, rows + (size_t)h * a.dim, a.ld, n, a.dim, a.silu);
+  lc_stage(Ks, kp, rows + hd + (size_t)h * a.dim, a.ld, n, a.dim, a.silu);
+  lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)hd + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
+  const float *S = a.chunk_state + (((size_t)c * a.heads + h) * a.dim) * a.vdim + v0;
+  for (int u = threadIdx.x; u < a.dim * (vc / 4); u += kLcThreads) {  // the state in three parts
+    const int r = u / (vc / 4), col = (u - r * (vc / 4)) * 4;
+    const float4 x = *reinterpret_cast<const float4 *>(S + (size_t)r * a.vdim + col);
+    uint32_t p0[kSplitParts], p1[kSplitParts];
+    split_pair(x.x, x.y, p0);
+    split_pair(x.z, x.w, p1);
+#pragma unroll
+    for (int p = 0; p < kSplitParts; ++p)
+      *reinterpret_cast<uint2 *>(Ss + (size_t)(p * a.dim + r) * kLcVPitch + col * 2) = make_uint2(p0[p], p1[p]);
+  }
+  __syncthreads();
+  const int m0 = warp * 16;
+  if (m0 >= n) return;  // no barrier follows
+  const uint32_t qs = (uint32_t)__cvta_generic_to_shared(smem), ks = (uint32_t)__cvta_generic_to_shared(Ks);
+  const uint32_t vs = (uint32_t)__cvta_generic_to_shared(Vs), ss = (uint32_t)__cvta_generic_to_shared(Ss);
+  float sc[kLinChunk / 8][4] = {}, acc[kLcCols / 8][4] = {};
+  for (int k0 = 0; k0 < a.dim; k0 += 16) {
+    uint32_t q0, q1, q2, q3;
+    ldsm4(frag_a(qs, m0, k0, kp, lane), q0, q1, q2, q3);
+#pragma unroll
+    for (int nt = 0; nt < kLinChunk / 8; nt += 2) {
+      if (nt * 8 <= m0 + 15) {  // later keys are invisible to every token of the warp
+        uint32_t b0, b1, b2, b3;
+        ldsm4(frag_b(ks, nt * 8, k0, kp, lane), b0, b1, b2, b3);
+        mma_bf16_16816(sc[nt], q0, q1, q2, q3, b0, b1);
+        mma_bf16_16816(sc[nt + 1], q0, q1, q2, q3, b2, b3);
+      }
+    }
+#pragma unroll
+    for (int nt = 0; nt < kLcCols / 8; nt += 2) {
+      if (nt * 8 < vc) {
+#pragma unroll
+        for (int p = 0; p < kSplitParts; ++p) {
+          uint32_t b0, b1, b2, b3;
+          ldsm4_t(frag_b_t(ss + p * a.dim * kLcVPitch, nt * 8, k0, kLcVPitch, lane), b0, b1, b2, b3);
+          mma_bf16_16816(acc[nt], q0, q1, q2, q3, b0, b1);
+          mma_bf16_16816(acc[nt + 1], q0, q1, q2, q3, b2, b3);
+        }
+      }
+    }
+  }
+  // the state's share decays by one step more than the token's place in the chunk
+  const float d_lo = s_pw[m0 + g + 1], d_hi = s_pw[m0 + g + 9];
+#pragma unroll
+  for (int nt = 0; nt < kLcCols / 8; ++nt) {
+    acc[nt][0] *= d_lo;
+    acc[nt][1] *= d_lo;
+    acc[nt][2] *= d_hi;
+    acc[nt][3] *= d_hi;
+  }
+  const int i_lo = m0 + g, i_hi = m0 + g + 8;
+#pragma unroll
+  for (int kk = 0; kk < kLinChunk / 16; ++kk) {
+    if (kk * 16 <= m0 + 15) {
+      uint32_t fa[4][kSplitParts];
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const float *s = sc[2 * kk + half];
+        const int j = kk * 16 + half * 8 + 2 * t;
+        const float w0 = j <= i_lo ? s[0] * a.k_scale * s_pw[i_lo - j] : 0.f, w1 = j + 1 <= i_lo ? s[1] * a.k_scale * s_pw[i_lo - j - 1] : 0.f;
+        const float w2 = j <= i_hi ? s[2] * a.k_scale * s_pw[i_hi - j] : 0.f, w3 = j + 1 <= i_hi ? s[3] * a.k_scale * s_pw[i_hi - j - 1] : 0.f;
+        split_pair(w0, w1, fa[2 * half]);
+        split_pair(w2, w3, fa[2 * half + 1]);
+      }
+#pragma unroll
+      for (int nt = 0; nt < kLcCols / 8; nt += 2) {
+        if (nt * 8 < vc) {
+          uint32_t b0, b1, b2, b3;
+          ldsm4_t(frag_b_t(vs, nt * 8, kk * 16, kLcVPitch, lane), b0, b1, b2, b3);
+#pragma unroll
+          for (int p = 0; p < kSplitParts; ++p) {
+            mma_bf16_16816(acc[nt], fa[0][p], fa[1][p], fa[2][p], fa[3][p], b0, b1);
+            mma_bf16_16816(acc[nt + 1], fa[0][p], fa[1][p], fa[2][p], fa[3][p], b2, b3);
+          }
+        }
+      }
+    }
+  }
+  const int hv = a.heads * a.vdim;
+  float *o = a.o + (size_t)c * kLinChunk * hv + (size_t)h * a.vdim + v0;
+#pragma unroll
+  for (int nt = 0; nt < kLcCols / 8; ++nt) {
+    if (nt * 8 < vc) {
+      const int col = nt * 8 + 2 * t;
+      if (i_lo < n) *reinterpret_cast<float2 *>(o + (size_t)i_lo * hv + col) = make_float2(acc[nt][0], acc[nt][1]);
+      if (i_hi < n) *reinterpret_cast<float2 *>(o + (size_t)i_hi * hv + col) = make_float2(acc[nt][2], acc[nt][3]);
+    }
+  }
+}
+
+// ---- norm over a head (or all heads), weight, gate ----
+template <typename Act>
+__global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNorm a) {
+  __shared__ float s_red[8];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n = a.heads * a.vdim;
+  const float *o = a.o + (size_t)blockIdx.x * n;
+  const Act *g = static_cast<const Act *>(a.g) + (size_t)blockIdx.x * a.ldg;
+  Act *out = static_cast<Act *>(a.out) + (size_t)blockIdx.x * a.ldo;
+  auto write = [&](int i, float scale) {
+    const float z = la_load(g + i), e = 1.0f / (1.0f + expf(-z));
+    const float v = o[i] * scale * (a.w ? a.w[i] : 1.f) * (a.gate == GATE_SILU ? z * e : e);
+    if constexpr (sizeof(Act) == 2) out[i] = f32_to_bf16_bits(v);
+    else out[i] = v;
+  };
+  if (a.per_head) {
+    for (int h = blockIdx.y * 8 + warp; h < a.heads; h += 8 * gridDim.y) {
+      float s = 0.f;
+      for (int i = lane; i < a.vdim; i += 32) s = fmaf(o[h * a.vdim + i], o[h * a.vdim + i], s);
+      const float scale = 1.0f / sqrtf(warp_sum(s) / (float)a.true_vdim + a.eps);
+      for (int i = lane; i < a.vdim; i += 32) write(h * a.vdim + i, scale);
+    }
+  } else {
+    float s = 0.f;
+    for (int i = tid * 4; i < n; i += 1024) {
+      const float4 v = *reinterpret_cast<const float4 *>(o + i);
+      s = fmaf(v.x, v.x, s), s = fmaf(v.y, v.y, s), s = fmaf(v.z, v.z, s), s = fmaf(v.w, v.w, s);
+    }
+    s = warp_sum(s);
+    if (lane == 0) s_red[warp] = s;
+    __syncthreads();
+    s = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) s += s_red[w];
+    const float scale = 1.0f / sqrtf(s / (float)(a.heads * a.true_vdim) + a.eps);
+    const int per = (n + gridDim.y - 1) / gridDim.y, end = min(n, (int)(blockIdx.y + 1) * per);
+    for (int i = blockIdx.y * per + tid; i < end; i += 256) write(i, scale);
+  }
+  if (blockIdx.y == 0)
+    for (int i = n + tid; i < a.ldo; i += 256) out[i] = Act(0);
+}
+
+int launch_gated_norm(const GatedNorm &a, int T, cudaStream_t stream) {
+  // few tokens: several CTAs share a token's heads (or columns; each then takes the whole sum)
+  const int parts = T >= sm_count() ? 1 : (a.per_head ? (a.heads + 7) / 8 : (a.heads * a.vdim + 1023) / 1024);
+  const dim3 grid(T, parts < 1 ? 1 : parts);
+  if (a.f32) gated_norm_kernel<float><<<grid, 256, 0, stream>>>(a);
+  else gated_norm_kernel<uint16_t><<<grid, 256, 0, stream>>>(a);
+  return launch_status("gated_norm_kernel");
+}
+
+static LaArgs la_args(const LinearAttn &a) {
+  LaArgs r{};
+  r.qkvg = a.qkvg;
+  r.decay_pow = a.decay_pow;
+  r.state = a.state;
+  r.o = a.o;
+  r.chunk_state = a.chunk_state;
+  r.heads = a.heads;
+  r.dim = a.dim;
+  r.vdim = a.vdim;
+  r.ld = a.ld;
+  r.silu = a.silu_qkv;
+  r.k_scale = a.k_scale;
+  return r;
+}
+
+template <typename Act>
+static int recurrent(const LaArgs &r, int seqs, cudaStream_t stream) {
+  const dim3 grid((r.vdim + 31) / 32, r.heads, seqs);
+  if (r.dim <= 64) linear_recurrent_kernel<Act, 2><<<grid, 256, 0, stream>>>(r);
+  else if (r.dim <= 128) linear_recurrent_kernel<Act, 4><<<grid, 256, 0, stream>>>(r);
+  else linear_recurrent_kernel<Act, 8><<<grid, 256, 0, stream>>>(r);
+  return launch_status("linear_recurrent_kernel");
+}
+
+static int check_shape(const LinearAttn &a) {
+  BLOK_REQUIRE(a.heads >= 1 && a.dim >= 16 && a.dim % 16 == 0 && a.dim <= kLinMaxDim && a.vdim >= 16 && a.vdim % 16 == 0 && a.ld % 8 == 0,
+               BLOK_ERR_SHAPE, "linear attention: %d heads of %d x %d (a head's key size is at most %d)", a.heads, a.dim, a.vdim, kLinMaxDim);
+  return BLOK_OK;
+}
+
+int launch_linear_step(const LinearAttn &a, const StackRows &rows, int B, cudaStream_t stream) {
+  if (int rc = check_shape(a)) return rc;
+  LaArgs r = la_args(a);
+  r.slot_of = rows.slot_of;
+  r.pos = rows.pos;
+  r.T = 1;
+  return a.f32 ? recurrent<float>(r, B, stream) : recurrent<uint16_t>(r, B, stream);
+}
+
+size_t linear_chunk_scratch_bytes(int heads, int dim, int vdim, int T) {
+  return (size_t)((T + kLinChunk - 1) / kLinChunk) * heads * dim * vdim * sizeof(float);
+}
+
+int launch_linear_chunk(const LinearAttn &a, int slot, long first_pos, int T, cudaStream_t stream) {
+  if (int rc = check_shape(a)) return rc;
+  LaArgs r = la_args(a);
+  r.slot = slot;
+  r.fresh = first_pos == 0;
+  r.T = T;
+  if (a.f32) return recurrent<float>(r, 1, stream);
+  if (T <= 8) return recurrent<uint16_t>(r, 1, stream);
+  r.chunks = (T + kLinChunk - 1) / kLinChunk;
+  const int kp = a.dim * 2 + 16;
+  const dim3 grid(r.chunks, a.heads, (a.vdim + kLcCols - 1) / kLcCols);
+  const size_t smem1 = (size_t)kSplitParts * kLinChunk * kp + (size_t)kLinChunk * kLcVPitch;
+  const size_t smem3 = (size_t)2 * kLinChunk * kp + (size_t)kLinChunk * kLcVPitch + (size_t)kSplitParts * a.dim * kLcVPitch;
+  BLOK_CUDA(cudaFuncSetAttribute(linear_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1));
+  BLOK_CUDA(cudaFuncSetAttribute(linear_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3));
+  linear_chunk_state_kernel<<<grid, kLcThreads, smem1, stream>>>(r);
+  if (int rc = launch_status("linear_chunk_state_kernel")) return rc;
+  linear_scan_kernel<<<dim3((a.dim * a.vdim / 4 + 127) / 128, a.heads), 128, 0, stream>>>(r);
+  if (int rc = launch_status("linear_scan_kernel")) return rc;
+  linear_chunk_out_kernel<<<grid, kLcThreads, smem3, stream>>>(r);
+  return launch_status("linear_chunk_out_kernel");
+}
+
+}  // namespace blok

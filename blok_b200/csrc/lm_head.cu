@@ -67,6 +67,38 @@ __global__ void argmax_bf16_kernel(const uint16_t *__restrict__ logits, int voca
   }
 }
 
+// The same over fp32 logits, rows `pitch` apart.
+__global__ void argmax_f32_kernel(const float *__restrict__ logits, int vocab, int pitch, uint32_t *__restrict__ ids) {
+  __shared__ float sv[32];
+  __shared__ int si[32];
+  const float *row = logits + (size_t)blockIdx.x * pitch;
+  float best = -INFINITY;
+  int bi = 0x7fffffff;
+  for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
+    const float v = row[i];
+    if (v > best) best = v, bi = i;
+  }
+  for (int pass = 0; pass < 2; ++pass) {
+#pragma unroll
+    for (int o = 16; o; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) best = ob, bi = oi;
+    }
+    if (pass == 1) break;
+    if ((threadIdx.x & 31) == 0) sv[threadIdx.x >> 5] = best, si[threadIdx.x >> 5] = bi;
+    __syncthreads();
+    if (threadIdx.x >= 32) return;
+    best = threadIdx.x < (blockDim.x >> 5) ? sv[threadIdx.x] : -INFINITY;
+    bi = threadIdx.x < (blockDim.x >> 5) ? si[threadIdx.x] : 0x7fffffff;
+  }
+  if (threadIdx.x == 0) ids[blockIdx.x] = bi == 0x7fffffff ? 0u : (uint32_t)bi;
+}
+int launch_argmax_f32(const float *logits, int vocab, int pitch, int T, uint32_t *ids, cudaStream_t stream) {
+  argmax_f32_kernel<<<T, 1024, 0, stream>>>(logits, vocab, pitch, ids);
+  return launch_status("argmax_f32_kernel");
+}
+
 // x[t, :] = table[ids[t], :]; an id outside the table raises *err (checked by the host wrapper's caller).
 __global__ void embed_kernel(const uint16_t *__restrict__ table, const uint32_t *__restrict__ ids, int vocab, int hidden,
                              uint16_t *__restrict__ x, unsigned *err) {

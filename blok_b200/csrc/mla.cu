@@ -19,6 +19,7 @@
 #include <new>
 
 #include "bf16_mma.cuh"
+#include "mla_merge.cuh"
 #include "wgemm.h"
 
 namespace blok {
@@ -31,55 +32,8 @@ int launch_bf16_gemv_splitk_pair(const uint16_t *w1, int rows1, uint16_t *y1, co
 int launch_bf16_gemv_splitk(const uint16_t *w, const uint16_t *x, uint16_t *y_bf16, float *y_f32, int rows, int cols, int T,
                             void *ws, size_t ws_bytes, cudaStream_t stream);
 
-// ---------------------------------------------------------------------------
-// Per-head mat-vec for up to 8 tokens: y[tok, head, r] = sum_c W[head][r][c] * x[tok, head, c].
-// grid = (rows/16, heads), 4 warps split K.  Strides are in elements.
-// ---------------------------------------------------------------------------
-__global__ void __launch_bounds__(128)
-    bf16_head_gemv_kernel(const uint16_t *__restrict__ w, long w_head_stride, const uint16_t *__restrict__ x,
-                          long x_tok_stride, long x_head_stride, uint16_t *__restrict__ y, long y_tok_stride,
-                          long y_head_stride, int cols, int T_all) {
-  extern __shared__ __align__(16) unsigned char smem[];
-  __shared__ float partial[4][16][8];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int g = lane >> 2, t = lane & 3;
-  const int head = blockIdx.y;
-  // blockIdx.z: the group of 8 tokens (the later groups find the head's matrix in L2)
-  const int T = min(8, T_all - 8 * (int)blockIdx.z);
-  x += (size_t)blockIdx.z * 8 * x_tok_stride;
-  y += (size_t)blockIdx.z * 8 * y_tok_stride;
-  const int per_row = cols / 8;
-  for (int u = tid; u < per_row * T; u += blockDim.x) {
-    int tok = u / per_row, c = u - tok * per_row;
-    uint4 v = reinterpret_cast<const uint4 *>(x + (size_t)tok * x_tok_stride + (size_t)head * x_head_stride)[c];
-    reinterpret_cast<uint4 *>(smem + tok * bf16_x_row_bytes(cols))[c] = v;
-  }
-  __syncthreads();
-  const size_t wrow = cols / 8;
-  const int row0 = blockIdx.x * 16;
-  const uint4 *w_lo = reinterpret_cast<const uint4 *>(w + (size_t)head * w_head_stride) + (size_t)(row0 + g) * wrow;
-  const uint4 *w_hi = w_lo + 8 * wrow;
-  const int tok = g < T ? g : T - 1;
-  const uint4 *xrow = reinterpret_cast<const uint4 *>(smem + tok * bf16_x_row_bytes(cols)) + t;
-  const int ksteps = cols / 32;
-  const int base = ksteps / 4, rem = ksteps % 4;
-  const int ks0 = warp * base + (warp < rem ? warp : rem);
-  const int nsteps = base + (warp < rem ? 1 : 0);
-  float d[4] = {0.f, 0.f, 0.f, 0.f};
-  bf16_rows16_accumulate(w_lo, w_hi, xrow, ks0, nsteps, t, d);
-  partial[warp][g][2 * t] = d[0];
-  partial[warp][g][2 * t + 1] = d[1];
-  partial[warp][g + 8][2 * t] = d[2];
-  partial[warp][g + 8][2 * t + 1] = d[3];
-  __syncthreads();
-  if (tid < 128) {
-    int r = tid >> 3, tk = tid & 7;
-    if (tk < T) {
-      float v = partial[0][r][tk] + partial[1][r][tk] + partial[2][r][tk] + partial[3][r][tk];
-      y[(size_t)tk * y_tok_stride + (size_t)head * y_head_stride + row0 + r] = f32_to_bf16_bits(v);
-    }
-  }
-}
+int launch_head_gemv(const uint16_t *w, long w_head_stride, const uint16_t *x, long x_tok_stride, long x_head_stride, uint16_t *y,
+                     long y_tok_stride, long y_head_stride, int rows, int cols, int heads, int T, cudaStream_t stream);
 
 // ---------------------------------------------------------------------------
 // Per sequence: RMSNorm of c_kv, RoPE of k_pe, append to the cache; RoPE of the
@@ -178,71 +132,6 @@ __global__ void transpose_wuk_kernel(const uint16_t *__restrict__ kv_b, uint16_t
   out[i] = kv_b[((size_t)h * (nope + v_head) + d) * kv_rank + j];
 }
 
-// ---------------------------------------------------------------------------
-// Merge of the split-KV partial results.  grid = (heads, B), 128 threads.
-//   part_o fp32 [B, splits, heads, kv_rank] unnormalised, part_ml fp32 [B, splits, heads, 2] = (max, sum)
-// ---------------------------------------------------------------------------
-__global__ void mla_merge_kernel(const float *__restrict__ part_o, const float *__restrict__ part_ml, int splits,
-                                 int heads, int kv_rank, uint16_t *__restrict__ o_lat) {
-  extern __shared__ float s_wt[];  // [splits] weight of every split: exp(m_s - M), 0 for an empty split
-  __shared__ float s_red[2][4];
-  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
-  const float *ml = part_ml + ((size_t)b * splits * heads + h) * 2;  // split s at + s * heads * 2
-  float M = -INFINITY;
-  for (int s = tid; s < splits; s += blockDim.x) M = fmaxf(M, ml[(size_t)s * heads * 2]);
-  M = warp_max(M);
-  if ((tid & 31) == 0) s_red[0][tid >> 5] = M;
-  __syncthreads();
-  M = fmaxf(fmaxf(s_red[0][0], s_red[0][1]), fmaxf(s_red[0][2], s_red[0][3]));
-  float L = 0.f;
-  for (int s = tid; s < splits; s += blockDim.x) {
-    const float m = ml[(size_t)s * heads * 2];
-    const float wt = m != -INFINITY ? expf(m - M) : 0.f;
-    s_wt[s] = wt;
-    L += wt * ml[(size_t)s * heads * 2 + 1];
-  }
-  L = warp_sum(L);
-  if ((tid & 31) == 0) s_red[1][tid >> 5] = L;
-  __syncthreads();
-  L = (s_red[1][0] + s_red[1][1]) + (s_red[1][2] + s_red[1][3]);
-  const float inv = L > 0.f ? 1.0f / L : 0.f;
-  const float *po = part_o + ((size_t)b * splits * heads + h) * kv_rank;  // split s at + s * heads * kv_rank
-  // four columns per thread, eight splits' worth of loads in flight per thread: the partial results (B x splits x 128 KB)
-  // come from L2 or HBM, and the kernel is as fast as it keeps bytes in flight.  Each column still adds its splits in
-  // ascending order.
-  const float4 *po4 = reinterpret_cast<const float4 *>(po);
-  const size_t stride4 = (size_t)heads * kv_rank / 4;
-  for (int j4 = tid; j4 < kv_rank / 4; j4 += blockDim.x) {
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    int s = 0;
-    for (; s + 8 <= splits; s += 8) {
-      float4 v[8];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) v[i] = __ldg(po4 + (size_t)(s + i) * stride4 + j4);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const float wt = s_wt[s + i];
-        acc.x = fmaf(wt, v[i].x, acc.x);
-        acc.y = fmaf(wt, v[i].y, acc.y);
-        acc.z = fmaf(wt, v[i].z, acc.z);
-        acc.w = fmaf(wt, v[i].w, acc.w);
-      }
-    }
-    for (; s < splits; ++s) {
-      const float4 v = __ldg(po4 + (size_t)s * stride4 + j4);
-      const float wt = s_wt[s];
-      acc.x = fmaf(wt, v.x, acc.x);
-      acc.y = fmaf(wt, v.y, acc.y);
-      acc.z = fmaf(wt, v.z, acc.z);
-      acc.w = fmaf(wt, v.w, acc.w);
-    }
-    uint2 o;
-    o.x = pack_bf16x2(acc.x * inv, acc.y * inv);
-    o.y = pack_bf16x2(acc.z * inv, acc.w * inv);
-    *reinterpret_cast<uint2 *>(o_lat + ((size_t)b * heads + h) * kv_rank + (size_t)j4 * 4) = o;
-  }
-}
-
 size_t mla_attend_smem_bytes();
 int launch_mla_attend(const uint16_t *q, const uint16_t *cache, long ctx_stride, const int *seq_len, int B, int splits,
                       float scale, float *part_o, float *part_ml, cudaStream_t stream);
@@ -256,15 +145,6 @@ int mla_attend_tc_trace(long long *host_out, int max_entries);
 int launch_mla_attend_paged(const uint16_t *q, const uint16_t *pool, const int *block_table, const int *slot_of,
                             int table_stride, int page_rows, const int *seq_len, int B, int splits, float scale,
                             float *part_o, float *part_ml, cudaStream_t stream);
-
-static int launch_head_gemv(const uint16_t *w, long w_head_stride, const uint16_t *x, long x_tok_stride,
-                            long x_head_stride, uint16_t *y, long y_tok_stride, long y_head_stride, int rows, int cols,
-                            int heads, int T, cudaStream_t stream) {
-  size_t smem = bf16_x_row_bytes(cols) * std::min(T, 8);
-  bf16_head_gemv_kernel<<<dim3(rows / 16, heads, (T + 7) / 8), 128, smem, stream>>>(w, w_head_stride, x, x_tok_stride, x_head_stride,
-                                                                      y, y_tok_stride, y_head_stride, cols, T);
-  return launch_status("bf16_head_gemv_kernel");
-}
 
 static size_t align256(size_t v) { return (v + 255) / 256 * 256; }
 

@@ -1,0 +1,149 @@
+// Kernels of the layer-stack models (model_stack.cu).  Sizes here are the padded ones the loader makes (zero rows and
+// columns), so that no kernel needs a bound on a head's dimensions; the true sizes enter only where a mean is taken.
+//
+// Activations are bf16, or fp32 for a BLOK_DTYPE_F32 model: `Act` pointers are void* with the flag `f32`.
+#pragma once
+#include <cuda_runtime.h>
+
+#include <cstdint>
+
+namespace blok {
+
+// Where a batch entry's cached rows and state live: entry i is the token at position pos[i] of the sequence in slot
+// slot_of[i].
+struct StackRows {
+  const int *slot_of = nullptr, *pos = nullptr;
+  const int *table = nullptr;  // [slots, table_stride] pages
+  int table_stride = 0, page_rows = 0;
+};
+
+// ---- residual streams (residual_streams.cu) ----
+constexpr int kMaxStreams = 16;
+struct StreamsStep {
+  int T = 0, width = 0, streams = 0;  // width: padded
+  float *x = nullptr;                 // [T, streams, width], updated in place
+  // x from the embedding (all streams alike) when ids is set
+  const uint32_t *ids = nullptr;
+  const uint16_t *embed = nullptr;  // bf16 [vocab, width]
+  int vocab = 0;
+  // else the update by a sublayer's output y: x'_t = sum_s mix[s, t] x_s + out[t] y with y = part_scale * the sum of
+  // `parts` rows: y_rows[part_at ? part_at[t * parts + k] : t * parts + k].  fp32 [., width]
+  const float *y_rows = nullptr;
+  int parts = 1;
+  const int *part_at = nullptr;
+  float part_scale = 1.f;
+  const float *mix = nullptr, *out = nullptr;
+  bool store_x = true;  // false: x stays as it was (the update feeds the norm only)
+  // what the next sublayer reads: u = sum_s in[s] x'_s (in NULL: the plain sum), h = tanh(alpha u) * w + b
+  const float *in = nullptr;
+  const float *norm_w = nullptr, *norm_b = nullptr;  // [width], zero in the padding; NULL: no norm wanted
+  float alpha = 0.f;
+  void *h = nullptr;  // Act [rows, width]
+  bool h_f32 = false;
+  int copies = 1;               // h of token t goes to rows copy_at[t * copies + k] (copy_at NULL: row t)
+  const int *copy_at = nullptr;
+  const int *rows = nullptr;    // only these tokens (T of them), row i of h is token rows[i]
+  float *sum = nullptr;         // fp32 [T, true_width]: the sum of the streams (for parity checks)
+  int true_width = 0;
+};
+int launch_streams_step(const StreamsStep &a, cudaStream_t stream);
+
+// ---- linear attention with a fixed decay per head (linear_attn.cu) ----
+enum { GATE_SILU = 0, GATE_SIGMOID = 1 };
+struct LinearAttn {
+  int heads = 0, dim = 0, vdim = 0;  // padded: multiples of 16
+  const void *qkvg = nullptr;        // Act [T, ld]: q | k | v | g, head by head
+  int ld = 0;
+  bool f32 = false;
+  bool silu_qkv = false;             // q, k and v go through SiLU (rounded to Act)
+  float k_scale = 1.f;
+  const float *decay_pow = nullptr;  // [heads, kLinChunk + 1]: decay^i
+  float *state = nullptr;            // fp32 [slots, heads, dim, vdim]
+  float *o = nullptr;                // fp32 [T, heads * vdim]
+  float *chunk_state = nullptr;      // scratch [chunks, heads, dim, vdim] of the chunked form
+};
+constexpr int kLinChunk = 64;
+constexpr int kLinMaxDim = 256;
+// One token of each of B sequences, or (chunk) T tokens of one sequence whose first position is first_pos.
+int launch_linear_step(const LinearAttn &a, const StackRows &r, int B, cudaStream_t stream);
+int launch_linear_chunk(const LinearAttn &a, int slot, long first_pos, int T, cudaStream_t stream);
+size_t linear_chunk_scratch_bytes(int heads, int dim, int vdim, int T);
+// out = rmsnorm(o) * w * gate(g): per head over true_vdim values (per_head), or over all heads together.
+struct GatedNorm {
+  int heads = 0, vdim = 0, true_vdim = 0;
+  bool per_head = false;
+  const float *w = nullptr;  // [heads * vdim] or NULL
+  float eps = 0.f;
+  int gate = GATE_SILU;
+  const float *o = nullptr;  // fp32 [T, heads * vdim]
+  const void *g = nullptr;   // Act [T, ldg]
+  int ldg = 0;
+  void *out = nullptr;       // Act [T, ldo], columns past heads * vdim zeroed
+  int ldo = 0;
+  bool f32 = false;
+};
+int launch_gated_norm(const GatedNorm &a, int T, cudaStream_t stream);
+
+// ---- latent attention over a paged cache of rows [latent | rotated key] (latent_attn.cu) ----
+struct LatentShape {
+  int heads = 0, dim = 0, rot = 0, vdim = 0, rank = 0, q_rank = 0;          // padded
+  int true_rot = 0, true_rank = 0, true_q_rank = 0, rot_dims = 0;
+  double rot_base = 1;
+  float scale = 1.f, eps = 0.f;
+  __host__ __device__ int row() const { return rank + rot; }  // a cached row
+  __host__ __device__ int head() const { return dim + rot; }  // a query head
+};
+// ckr fp32 [T, q_rank + row]: the query latent is normed into cq (Act [T, q_rank]); the key latent is normed, the shared
+// key part rotated, and the row appended to the pool (Act [pages, page_rows, row]).
+int launch_latent_append(const LatentShape &s, const float *ckr, const float *q_norm, const float *kv_norm, const StackRows &r, int T, void *cq,
+                         void *pool, bool f32, cudaStream_t stream);
+// Rotates the last `rot` columns of every query head of q (Act [T, heads, head()]) into dst, whose heads are dst_head
+// columns apart starting at dst_off (dst == q, dst_head == head(), dst_off == dim: in place).
+int launch_latent_rotate(const LatentShape &s, const void *q, const StackRows &r, int T, void *dst, int dst_head, int dst_off, bool f32,
+                         cudaStream_t stream);
+// Absorbed form: q_abs Act [T, heads, row()], o Act [T, heads, rank].  Entry i attends to positions 0..pos[i].
+// Scratch for calls of up to T entries: part_o fp32 [max_parts, heads, rank] and part_ml fp32 [max_parts, heads, 2].  Each
+// buffer must hold finite values (part_o) at the first call and serve this purpose only: an empty part leaves its rows as
+// they were and the merge multiplies them by zero.
+size_t latent_attend_max_parts(const LatentShape &s, int T, long max_ctx);
+int launch_latent_attend(const LatentShape &s, const void *q_abs, const void *pool, const StackRows &r, int T, long max_ctx, void *o, bool f32,
+                         float *part_o, float *part_ml, cudaStream_t stream);
+// Prompt form (bf16): the first n cached rows of the sequence in `slot` copied to c_all [n, rank] and kr_all [n, rot] ...
+int launch_latent_gather(const LatentShape &s, const uint16_t *pool, const StackRows &r, int slot, int n, uint16_t *c_all, uint16_t *kr_all,
+                         cudaStream_t stream);
+// ... and, with kv = the per-head keys and values made from them (bf16 [n, heads * (dim + vdim)]: all keys, then all
+// values), causal attention of T queries at positions n - T .. n - 1: q bf16 [T, heads, head()], o bf16 [T, ldo].
+bool latent_prompt_supports(const LatentShape &s);
+int launch_latent_prompt(const LatentShape &s, const uint16_t *q, const uint16_t *kv, const uint16_t *kr_all, int T, int n, uint16_t *o, int ldo,
+                         cudaStream_t stream);
+
+// ---- experts chosen by a table of token ids (table_experts.cu) ----
+struct ExpertPlan {          // of one layer and call
+  int *at = nullptr;         // [T * top] row of assignment (t, k) in expert order
+  int *tile_expert = nullptr, *tile_start = nullptr, *tile_count = nullptr, *num_tiles = nullptr;  // tiles of up to 128 rows
+};
+struct ExpertPlanArgs {
+  const int *table = nullptr;  // [vocab, top]
+  int experts = 0, top = 0;
+  ExpertPlan plan;
+};
+constexpr int kMaxTableExperts = 4096;
+int expert_plan_max_tiles(int assignments, int experts);
+// One block per layer of `layers` (device array of n_layers).
+int launch_expert_plan(const ExpertPlanArgs *layers, int n_layers, const uint32_t *ids, int vocab, int T, cudaStream_t stream);
+// y[a, :] = act(W[e(a)] x[row(a), :]) assignment by assignment, e(a) = table[ids[a / top]][a % top] and row(a) = a / top
+// (shared_x) or a.  W bf16 [experts, R, K]; x Act [., K]; y Act or fp32 [T * top, R].
+int launch_expert_gemv(const uint16_t *w, int R, int K, const int *table, const uint32_t *ids, int vocab, int top, int T, const void *x, bool x_f32,
+                       bool shared_x, bool relu2, void *y, bool y_f32, cudaStream_t stream);
+
+// ---- fp32 products (gemm_f32.cu): y[z][t, r] = sum_k x[z][t, k] W[z][r, k], W bf16, x and y fp32 ----
+struct GemmF32 {
+  const uint16_t *w = nullptr;
+  const float *x = nullptr;
+  float *y = nullptr;
+  int R = 0, K = 0, T = 0, ldw = 0, ldx = 0, ldy = 0, batch = 1;
+  long w_stride = 0, x_stride = 0, y_stride = 0;  // between batches
+};
+int launch_gemm_f32(const GemmF32 &g, cudaStream_t stream);
+
+}  // namespace blok

@@ -193,52 +193,6 @@ __global__ void __launch_bounds__(kWgThreads) wgemm_kernel(const WgArgs a) {
   }
 }
 
-// Adds the K-split partial sums in split order and applies the epilogue of wgemm_kernel.  grid = (ceil(R / 256), n_rows).
-template <bool SWIGLU>
-__global__ void wgemm_splitk_reduce_kernel(const WgArgs a, int nz) {
-  const int p = blockIdx.y, row = blockIdx.x * blockDim.x + threadIdx.x;
-  if (row >= a.R) return;
-  const int cols = SWIGLU ? 2 * a.R : a.R;
-  const float *ps = a.splitk_ws + (size_t)p * cols + row;
-  const size_t stride = (size_t)a.n_rows * cols;
-  float v = 0.f, u = 0.f;
-  for (int z = 0; z < nz; ++z) {
-    v += ps[z * stride];
-    if (SWIGLU) u += ps[z * stride + a.R];
-  }
-  const size_t o = (a.out_index ? (size_t)a.out_index[p] : (size_t)p) * a.R + row;
-  if (SWIGLU) {
-    const float gv = round_bf16(v), uv = round_bf16(u);
-    a.out_bf16[o] = f32_to_bf16_bits(round_bf16(round_bf16(gv / (1.0f + expf(-gv))) * uv));
-  } else if (a.out_f32) {
-    a.out_f32[o] = v;
-  } else {
-    a.out_bf16[o] = f32_to_bf16_bits(v);
-  }
-}
-
-int wgemm_splitk_factor(int mode, int K, int R, int tiles) {
-  if (mode != WG_BF16_PLAIN && mode != WG_BF16_SWIGLU) return 1;
-  const int rows_per_cta = mode == WG_BF16_SWIGLU ? 8 * kWgWarps : 16 * kWgWarps;
-  if (R % rows_per_cta || K % kWgChunk || tiles < 1) return 1;
-  const int ctas = R / rows_per_cta * tiles, chunks = K / kWgChunk;
-  return std::max(1, std::min(chunks, 2 * sm_count() / ctas));
-}
-size_t wgemm_splitk_bytes(int mode, int K, int R, int max_rows) {
-  size_t worst = 0;
-  {  // the weight-streaming kernel over up to kWgStreamTokens rows
-    const int nz = wgemm_stream_split(mode, K, R);
-    if (nz > 1) worst = (size_t)nz * std::min(max_rows, kWgStreamTokens) * (mode == WG_BF16_SWIGLU ? 2 * R : R) * sizeof(float);
-  }
-  for (int tiles = 1; tiles <= (max_rows + kWgTokens - 1) / kWgTokens; ++tiles) {
-    const int nz = wgemm_splitk_factor(mode, K, R, tiles);
-    if (nz <= 1) break;  // the factor falls as the tiles grow in number
-    const size_t rows = (size_t)std::min(max_rows, tiles * kWgTokens);
-    worst = std::max(worst, (size_t)nz * rows * (mode == WG_BF16_SWIGLU ? 2 * R : R) * sizeof(float));
-  }
-  return worst;
-}
-
 size_t wgemm_smem_bytes() { return (size_t)kWgTokens * kWgTokPitch; }
 
 // 0 = pick by size, 1 = mma.sync kernel always, 2 = tcgen05 kernels wherever they apply
@@ -267,13 +221,7 @@ int launch_wgemm(int mode, const WgArgs &args_in, int max_tiles, cudaStream_t st
   if (!i4 && forced == 0 && wgemm_stream_supports(mode, args)) {
     int nz = 1;
     if (int rc = launch_wgemm_stream(mode, args, &nz, stream)) return rc;
-    if (nz > 1) {
-      const dim3 rg((args.R + 255) / 256, args.n_rows);
-      if (swiglu) wgemm_splitk_reduce_kernel<true><<<rg, 256, 0, stream>>>(args, nz);
-      else wgemm_splitk_reduce_kernel<false><<<rg, 256, 0, stream>>>(args, nz);
-      return launch_status("wgemm_splitk_reduce_kernel");
-    }
-    return BLOK_OK;
+    return nz > 1 ? launch_wgemm_splitk_reduce(mode, args, nz, stream) : BLOK_OK;
   }
   // bf16: the tcgen05 kernel's 256-token tiles leave most SMs idle below about 650 tokens (shared expert: 376 us from
   // 128 to 1,024 tokens, against 106 / 162 / 297 / 585 us for the K-split mma.sync kernel at 128 / 256 / 512 / 1,024)
@@ -301,33 +249,7 @@ int launch_wgemm(int mode, const WgArgs &args_in, int max_tiles, cudaStream_t st
   }
 #undef BLOK_WG_LAUNCH
   if (int rc = launch_status("wgemm_kernel")) return rc;
-  if (grid.z > 1) {
-    const dim3 rg((args.R + 255) / 256, args.n_rows);
-    if (swiglu) wgemm_splitk_reduce_kernel<true><<<rg, 256, 0, stream>>>(args, (int)grid.z);
-    else wgemm_splitk_reduce_kernel<false><<<rg, 256, 0, stream>>>(args, (int)grid.z);
-    return launch_status("wgemm_splitk_reduce_kernel");
-  }
-  return BLOK_OK;
-}
-
-int launch_wgemm_rows(int mode, const void *w_a, const void *w_b, const uint16_t *x, uint16_t *out_bf16, float *out_f32, int R, int K,
-                      int T, float *splitk_ws, size_t splitk_bytes, cudaStream_t stream) {
-  WgArgs r;
-  r.w_a = w_a; r.w_b = w_b; r.s_a = r.s_b = nullptr; r.expert_stride_rows = 0; r.x = x; r.x_index = nullptr;
-  r.K = K; r.R = R; r.out_bf16 = out_bf16; r.out_f32 = out_f32;
-  r.tile_expert = r.tile_start = r.tile_count = r.num_tiles = nullptr; r.out_index = nullptr;
-  r.identity_tiles = 1; r.n_rows = T; r.splitk_ws = splitk_ws; r.splitk_bytes = splitk_bytes;
-  BLOK_REQUIRE(wgemm_stream_supports(mode, r), BLOK_ERR_SHAPE, "wgemm rows: %d rows x %d columns over %d tokens is outside the streaming kernel",
-               R, K, T);
-  int nz = 1;
-  if (int rc = launch_wgemm_stream(mode, r, &nz, stream)) return rc;
-  if (nz > 1) {
-    const dim3 rg((R + 255) / 256, T);
-    if (mode == WG_BF16_SWIGLU) wgemm_splitk_reduce_kernel<true><<<rg, 256, 0, stream>>>(r, nz);
-    else wgemm_splitk_reduce_kernel<false><<<rg, 256, 0, stream>>>(r, nz);
-    return launch_status("wgemm_splitk_reduce_kernel");
-  }
-  return BLOK_OK;
+  return grid.z > 1 ? launch_wgemm_splitk_reduce(mode, args, (int)grid.z, stream) : BLOK_OK;
 }
 
 }  // namespace blok

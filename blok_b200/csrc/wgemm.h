@@ -68,6 +68,8 @@ int launch_wgemv_small(int mode, const WgArgs &args, cudaStream_t stream);
 // wait in args.splitk_ws for wgemm_splitk_reduce_kernel (launch_wgemm runs it).  wgemm_stream_split: the split of a shape.
 bool wgemm_stream_supports(int mode, const WgArgs &args);
 int wgemm_stream_split(int mode, int K, int R);
+// The reduction behind a K-split launch: adds the nz partial sums in split order and applies the epilogue.
+int launch_wgemm_splitk_reduce(int mode, const WgArgs &args, int nz, cudaStream_t stream);
 int launch_wgemm_stream(int mode, const WgArgs &args, int *splits, cudaStream_t stream);
 // One dense product through launch_wgemm without tile tables: out[T, R] = W[R, K] x[T, K] (mode WG_BF16_PLAIN; bf16 or
 // fp32 output) or the SwiGLU front half of (w_a = gate, w_b = up) (mode WG_BF16_SWIGLU), for 1 <= T <= kWgStreamTokens.

@@ -203,4 +203,72 @@ int launch_wgemm_stream(int mode, const WgArgs &args, int *splits, cudaStream_t 
   return launch_status("wgemm_stream_kernel");
 }
 
+// Adds the K-split partial sums in split order and applies the epilogue of the GEMM kernels.  grid = (ceil(R / 256), n_rows).
+template <bool SWIGLU>
+__global__ void wgemm_splitk_reduce_kernel(const WgArgs a, int nz) {
+  const int p = blockIdx.y, row = blockIdx.x * blockDim.x + threadIdx.x;
+  if (row >= a.R) return;
+  const int cols = SWIGLU ? 2 * a.R : a.R;
+  const float *ps = a.splitk_ws + (size_t)p * cols + row;
+  const size_t stride = (size_t)a.n_rows * cols;
+  float v = 0.f, u = 0.f;
+  for (int z = 0; z < nz; ++z) {
+    v += ps[z * stride];
+    if (SWIGLU) u += ps[z * stride + a.R];
+  }
+  const size_t o = (a.out_index ? (size_t)a.out_index[p] : (size_t)p) * a.R + row;
+  if (SWIGLU) {
+    const float gv = round_bf16(v), uv = round_bf16(u);
+    a.out_bf16[o] = f32_to_bf16_bits(round_bf16(round_bf16(gv / (1.0f + expf(-gv))) * uv));
+  } else if (a.out_f32) {
+    a.out_f32[o] = v;
+  } else {
+    a.out_bf16[o] = f32_to_bf16_bits(v);
+  }
+}
+
+int launch_wgemm_splitk_reduce(int mode, const WgArgs &args, int nz, cudaStream_t stream) {
+  const dim3 rg((args.R + 255) / 256, args.n_rows);
+  if (mode == WG_BF16_SWIGLU || mode == WG_I4_SWIGLU) wgemm_splitk_reduce_kernel<true><<<rg, 256, 0, stream>>>(args, nz);
+  else wgemm_splitk_reduce_kernel<false><<<rg, 256, 0, stream>>>(args, nz);
+  return launch_status("wgemm_splitk_reduce_kernel");
+}
+
+// The mma.sync kernel (wgemm.cu) has 128 weight rows per CTA (64 + 64 for SwiGLU) and splits whole 512-column chunks.
+int wgemm_splitk_factor(int mode, int K, int R, int tiles) {
+  if (mode != WG_BF16_PLAIN && mode != WG_BF16_SWIGLU) return 1;
+  const int rows_per_cta = mode == WG_BF16_SWIGLU ? 64 : 128;
+  if (R % rows_per_cta || K % 512 || tiles < 1) return 1;
+  const int ctas = R / rows_per_cta * tiles, chunks = K / 512;
+  return std::max(1, std::min(chunks, 2 * sm_count() / ctas));
+}
+size_t wgemm_splitk_bytes(int mode, int K, int R, int max_rows) {
+  size_t worst = 0;
+  {  // the weight-streaming kernel over up to kWgStreamTokens rows
+    const int nz = wgemm_stream_split(mode, K, R);
+    if (nz > 1) worst = (size_t)nz * std::min(max_rows, kWgStreamTokens) * (mode == WG_BF16_SWIGLU ? 2 * R : R) * sizeof(float);
+  }
+  for (int tiles = 1; tiles <= (max_rows + kWgTileTokens - 1) / kWgTileTokens; ++tiles) {
+    const int nz = wgemm_splitk_factor(mode, K, R, tiles);
+    if (nz <= 1) break;  // the factor falls as the tiles grow in number
+    const size_t rows = (size_t)std::min(max_rows, tiles * kWgTileTokens);
+    worst = std::max(worst, (size_t)nz * rows * (mode == WG_BF16_SWIGLU ? 2 * R : R) * sizeof(float));
+  }
+  return worst;
+}
+
+int launch_wgemm_rows(int mode, const void *w_a, const void *w_b, const uint16_t *x, uint16_t *out_bf16, float *out_f32, int R, int K,
+                      int T, float *splitk_ws, size_t splitk_bytes, cudaStream_t stream) {
+  WgArgs r;
+  r.w_a = w_a; r.w_b = w_b; r.s_a = r.s_b = nullptr; r.expert_stride_rows = 0; r.x = x; r.x_index = nullptr;
+  r.K = K; r.R = R; r.out_bf16 = out_bf16; r.out_f32 = out_f32;
+  r.tile_expert = r.tile_start = r.tile_count = r.num_tiles = nullptr; r.out_index = nullptr;
+  r.identity_tiles = 1; r.n_rows = T; r.splitk_ws = splitk_ws; r.splitk_bytes = splitk_bytes;
+  BLOK_REQUIRE(wgemm_stream_supports(mode, r), BLOK_ERR_SHAPE, "wgemm rows: %d rows x %d columns over %d tokens is outside the streaming kernel",
+               R, K, T);
+  int nz = 1;
+  if (int rc = launch_wgemm_stream(mode, r, &nz, stream)) return rc;
+  return nz > 1 ? launch_wgemm_splitk_reduce(mode, r, nz, stream) : BLOK_OK;
+}
+
 }  // namespace blok

@@ -14,7 +14,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "libblok_b200.so")
 
 OK = 0
-ABI_VERSION = 3  # BLOK_ABI_VERSION of include/blok_b200.h: the layout of the structures mirrored below
+ABI_VERSION = 4  # BLOK_ABI_VERSION of include/blok_b200.h: the layout of the structures mirrored below
 
 
 class BlokError(RuntimeError):
@@ -726,8 +726,72 @@ def _rt():
     return _cudart
 
 
+class ModelOptions(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("dtype", "max_batch", "max_ctx", "prefill_chunk", "kv_page_rows", "kv_pages")] + [("eos_id", C.c_uint32)]
+
+
+def architectures():
+    """Names of the architectures that Model.open can read from a config.json."""
+    f = load().blok_model_architectures
+    f.restype = C.c_char_p
+    return f().decode().split()
+
+
 class Model:
-    """The whole decode model with seeded synthetic weights (generate(), src/kimi_exec.cu:780-893)."""
+    """The whole decode model with seeded synthetic weights (generate(), src/kimi_exec.cu:780-893), or a model described by
+    a config.json (Model.open, Model.open_synthetic)."""
+
+    @classmethod
+    def open(cls, directory, dtype="bfloat16", **options):
+        """The model of a folder with config.json and model.safetensors (blok_model_open)."""
+        return cls._opened(lambda o, h: load().blok_model_open(str(directory).encode(), o, h), dtype, options)
+
+    @classmethod
+    def open_synthetic(cls, config, seed=1, dtype="bfloat16", **options):
+        """A model of the given configuration (a dict) with seeded weights (blok_model_open_synthetic)."""
+        import json
+        text = json.dumps(config).encode()
+        return cls._opened(lambda o, h: load().blok_model_open_synthetic(text, C.c_uint64(seed), o, h), dtype, options)
+
+    @classmethod
+    def _opened(cls, call, dtype, options):
+        lib = load()
+        opt = ModelOptions()
+        lib.blok_model_default_options(C.byref(opt))
+        opt.dtype = {"bfloat16": 0, "float32": 1}[dtype]
+        for k, v in options.items():
+            if not hasattr(opt, k):
+                raise BlokError(-1, "unknown model option %r" % k)
+            setattr(opt, k, v)
+        self = cls.__new__(cls)
+        self._handle = C.c_void_p()
+        _check(call(C.byref(opt), C.byref(self._handle)))
+        self.cfg = ModelConfig()
+        _check(lib.blok_model_get_config(self._handle, C.byref(self.cfg)))
+        return self
+
+    def extend(self, slot, tokens, want=()):
+        """The next tokens (host list) of the sequence in `slot`; the logits at the places `want` among them, a numpy fp32
+        array [len(want), vocab] (blok_model_extend_slot)."""
+        import numpy as np
+        ids = np.ascontiguousarray(tokens, np.uint32)
+        places = np.ascontiguousarray(want, np.int32)
+        out = np.empty((places.size, self.cfg.vocab), np.float32)
+        _check(load().blok_model_extend_slot(self._handle, C.c_int(slot), ids.ctypes.data_as(C.c_void_p), C.c_int(ids.size),
+                                             places.ctypes.data_as(C.c_void_p), C.c_int(places.size), out.ctypes.data_as(C.c_void_p),
+                                             _stream()))
+        return out
+
+    def trace_layers(self, max_rows):
+        """From now on calls of up to max_rows tokens store the residual after every layer run: the device tensor
+        [layer runs, max_rows, hidden] they are stored in (blok_model_trace_layers).  0 ends it."""
+        runs = C.c_int()
+        _check(load().blok_model_trace_layers(self._handle, None, C.c_int(0), C.byref(runs)))
+        if not max_rows:
+            return None
+        self._trace = torch.zeros((runs.value, max_rows, self.cfg.hidden), dtype=torch.float32, device="cuda")
+        _check(load().blok_model_trace_layers(self._handle, _ptr(self._trace), C.c_int(max_rows), C.byref(runs)))
+        return self._trace
 
     def __init__(self, seed=4, **overrides):
         lib = load()

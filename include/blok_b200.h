@@ -46,8 +46,9 @@ enum {
 };
 
 /* 2: blok_model_config gained prefill_chunk, kv_page_rows and kv_pages (appended).
- * 3: blok_comm_*, blok_moe_ep_*, blok_model_set_comm; blok_model_config gained ep_rank and ep_world (appended). */
-#define BLOK_ABI_VERSION 3
+ * 3: blok_comm_*, blok_moe_ep_*, blok_model_set_comm; blok_model_config gained ep_rank and ep_world (appended).
+ * 4: blok_model_open, blok_model_open_synthetic, blok_model_extend_slot, blok_model_trace_layers. */
+#define BLOK_ABI_VERSION 4
 
 /* Message of the last failure on this thread ("" if none). */
 const char *blok_last_error(void);
@@ -539,6 +540,44 @@ void blok_model_default_config(blok_model_config *cfg);
  * weights 1).  Stands in for the checkpoint loader of the reference (:736-778). */
 int blok_model_create_synthetic(const blok_model_config *cfg, uint64_t seed, blok_model_t **out);
 int blok_model_destroy(blok_model_t *model);
+
+/* Models described by a config.json.  The library keeps a registry of architectures; "architecture" of config.json
+ * picks one.  blok_model_architectures: their names, separated by spaces.
+ *   Nomozen: a decoder of retention, lightning and latent-attention layers with table-routed squared-ReLU experts,
+ *            Dynamic-Tanh norms and hyper-connected residual streams (csrc/nomozen.cu).
+ * Such a model is always paged; slots, steps, prompts, generation and batching are the calls below, as for every model. */
+enum { BLOK_DTYPE_BF16 = 0, /* products and activations in bf16, fp32 accumulation; norms, scores, decays, recurrent states,
+                               positions and the residual in fp32 */
+       BLOK_DTYPE_F32 = 1   /* everything in fp32 (the weights are bf16 values) */ };
+typedef struct blok_model_options {
+  int dtype;         /* BLOK_DTYPE_BF16 */
+  int max_batch;     /* sequence slots, 1..64 */
+  int max_ctx;       /* tokens per sequence */
+  int prefill_chunk; /* tokens of a prompt per pass */
+  int kv_page_rows;  /* rows per cache page, a multiple of 32 */
+  int kv_pages;      /* pages of the pool; 0: enough for max_batch sequences of max_ctx tokens */
+  uint32_t eos_id;   /* ends a generation; 0xffffffff: none */
+} blok_model_options;
+const char *blok_model_architectures(void);
+/* bf16, 1 slot, max_ctx 4096, chunks of 1024 tokens, pages of 64 rows, no end-of-sequence id. */
+void blok_model_default_options(blok_model_options *options);
+/* Reads dir/config.json and dir/model.safetensors.  options NULL: the defaults.  A missing tensor, or one of another type
+ * or shape than the configuration asks for, is an error that names it. */
+int blok_model_open(const char *dir, const blok_model_options *options, blok_model_t **out);
+/* The same from the text of a config.json, with seeded weights made on the device. */
+int blok_model_open_synthetic(const char *config_json, uint64_t seed, const blok_model_options *options, blok_model_t **out);
+
+/* The next n tokens (HOST ids) of the sequence in `slot`, and the logits at some of them: want[i] (HOST, n_want of them,
+ * each in [0, n)) names a place among these tokens, logits (HOST, fp32 [n_want, vocab]) receives its row.  One token goes
+ * through the decode step, more through the prompt path in chunks.  Nothing is sampled.  Synchronises `stream` when
+ * something is wanted.  Only models opened from a config.json offer it. */
+int blok_model_extend_slot(blok_model_t *model, int slot, const uint32_t *ids, int n, const int *want, int n_want,
+                           float *logits, blok_stream_t stream);
+
+/* For parity checks: from now on every call of at most max_rows tokens stores the residual (the sum of the streams) after
+ * every layer run in `buffer` (DEVICE, fp32 [layer runs, max_rows, hidden]; a looped layer counts each time).  Steps then
+ * run eagerly.  NULL ends it.  *runs receives the number of layer runs. */
+int blok_model_trace_layers(blok_model_t *model, float *buffer, int max_rows, int *runs);
 
 /* Device pointer and byte size of a weight tensor, for tests and loaders.  layer = -1
  * for "embed_tokens", "norm", "lm_head"; per layer: "input_layernorm",
