@@ -5,6 +5,8 @@
 //                  [--synthetic-seed <s>] [--layers <n>] [--experts <n>] [--vocab <n>] [--max-ctx <n>]
 //                  [--hidden --inter --dense-inter --shared-inter --heads --q-rank --kv-rank <n>]
 //                  [--prefill-chunk <n>]   prompt in chunks of n tokens (1..64) instead of token by token
+//   blok-kimi-exec --model <dir> --prompt-tokens <id,id,...> --tokens <n> [--dtype bfloat16|float32] [--max-ctx <n>]
+//                  [--prefill-chunk <n>]   a model described by config.json, with model.safetensors beside it
 //
 // Success: exit 0 and exactly one stdout line {"status":"ok","token_ids":[...]}.
 // Failure: a message on stderr and exit 1, which blok/runtime.py:86-94 turns into
@@ -13,6 +15,7 @@
 // names into the model's resident tensors on the current GPU (the model must fit that
 // GPU: the size flags exist for reduced checkpoints and tests).  With --synthetic-seed
 // the index is not read and the weights are seeded synthetic tensors of the requested size.
+#include <algorithm>
 #include <charconv>
 #include <cstdint>
 #include <cstdio>
@@ -39,9 +42,9 @@ unsigned long long parse_number(std::string_view text, const char *what) {
 }
 
 struct Options {
-  std::string index, prompt;
+  std::string index, prompt, model;
   unsigned long long tokens = 0, seed = 0;
-  bool synthetic = false;
+  bool synthetic = false, f32 = false;
   blok_model_config cfg;
 };
 
@@ -68,7 +71,11 @@ Options parse_command_line(int argc, char **argv) {
     if (flag.substr(0, 2) != "--") throw Fail{"unknown flag: " + std::string(flag)};
     const std::string_view name = flag.substr(2);
     if (name == "index") o.index = value;
-    else if (name == "prompt-tokens") o.prompt = value;
+    else if (name == "model") o.model = value;
+    else if (name == "dtype") {
+      if (value != "bfloat16" && value != "float32") throw Fail{"unknown dtype: " + std::string(value)};
+      o.f32 = value == "float32";
+    } else if (name == "prompt-tokens") o.prompt = value;
     else if (name == "tokens") o.tokens = parse_number(value, "tokens");
     else if (name == "synthetic-seed") o.seed = parse_number(value, "synthetic-seed"), o.synthetic = true;
     else {
@@ -79,7 +86,7 @@ Options parse_command_line(int argc, char **argv) {
       o.cfg.*(hit->field) = (int)parse_number(value, hit->name);
     }
   }
-  if ((o.index.empty() && !o.synthetic) || o.prompt.empty() || o.tokens == 0) throw Fail{"bad args"};
+  if ((o.index.empty() && o.model.empty() && !o.synthetic) || o.prompt.empty() || o.tokens == 0) throw Fail{"bad args"};
   return o;
 }
 
@@ -103,17 +110,33 @@ void require_ok(int rc, const char *stage) {
   if (rc != BLOK_OK) throw Fail{std::string(stage) + ": " + blok_last_error()};
 }
 
+// The model of a folder with a config.json (its vocabulary bounds the prompt when it generates).
+blok_model_t *open_folder(const Options &o, size_t n_prompt) {
+  blok_model_options opt;
+  blok_model_default_options(&opt);
+  opt.dtype = o.f32 ? BLOK_DTYPE_F32 : BLOK_DTYPE_BF16;
+  opt.max_ctx = std::max(o.cfg.max_ctx, (int)(n_prompt + o.tokens));
+  if (o.cfg.prefill_chunk) opt.prefill_chunk = o.cfg.prefill_chunk;
+  blok_model_t *model = nullptr;
+  require_ok(blok_model_open(o.model.c_str(), &opt, &model), "model");
+  return model;
+}
+
 int run(int argc, char **argv) {
   Options o = parse_command_line(argc, argv);
-  const std::vector<uint32_t> prompt = parse_prompt(o.prompt, o.cfg.vocab);
-  if ((unsigned long long)o.cfg.max_ctx < prompt.size() + o.tokens) o.cfg.max_ctx = (int)(prompt.size() + o.tokens);
-  // --synthetic-seed stands in for the checkpoint: the index is then not read.  Otherwise the index is parsed and
-  // checked against the forward contract before any device memory is taken.
-  if (!o.synthetic) require_ok(blok_index_validate(o.index.c_str(), &o.cfg, nullptr, nullptr), "index");
+  const std::vector<uint32_t> prompt = parse_prompt(o.prompt, o.model.empty() ? o.cfg.vocab : INT32_MAX);
   blok_model_t *model = nullptr;
-  require_ok(blok_model_create_synthetic(&o.cfg, o.seed, &model), "model");
-  // every tensor of the forward contract is read once into the model's resident tensors
-  if (!o.synthetic) require_ok(blok_model_load_index(model, o.index.c_str()), "index");
+  if (!o.model.empty()) {
+    model = open_folder(o, prompt.size());
+  } else {
+    if ((unsigned long long)o.cfg.max_ctx < prompt.size() + o.tokens) o.cfg.max_ctx = (int)(prompt.size() + o.tokens);
+    // --synthetic-seed stands in for the checkpoint: the index is then not read.  Otherwise the index is parsed and
+    // checked against the forward contract before any device memory is taken.
+    if (!o.synthetic) require_ok(blok_index_validate(o.index.c_str(), &o.cfg, nullptr, nullptr), "index");
+    require_ok(blok_model_create_synthetic(&o.cfg, o.seed, &model), "model");
+    // every tensor of the forward contract is read once into the model's resident tensors
+    if (!o.synthetic) require_ok(blok_model_load_index(model, o.index.c_str()), "index");
+  }
   std::vector<uint32_t> generated(o.tokens);
   int n = 0;
   require_ok(blok_model_generate(model, prompt.data(), (int)prompt.size(), (int)o.tokens, generated.data(), &n), "generate");

@@ -77,6 +77,7 @@ extern "C" int blok_model_destroy(blok_model_t *m) {
     if (g) cudaGraphExecDestroy(g);
   blok_kv_pages_destroy(m->pages);
   if (m->family) m->family->destroy(m);
+  if (m->own_stream) cudaStreamDestroy(m->own_stream);
   cudaError_t first = cudaSuccess;
   for (void *p : m->allocations) {
     cudaError_t e = cudaFree(p);
@@ -408,6 +409,14 @@ extern "C" long blok_model_slot_length(blok_model_t *m, int slot) {
 
 extern "C" int blok_model_free_pages(blok_model_t *m) { return (m && m->pages) ? blok_kv_pages_free_count(m->pages) : -1; }
 
+// The stream generation runs on.  It is a blocking stream: copies and memsets on the legacy default stream are ordered with
+// it.
+static int generation_stream(blok_model_t *m, blok_stream_t *out) {
+  if (!m->own_stream) BLOK_CUDA(cudaStreamCreate(&m->own_stream));
+  *out = (blok_stream_t)m->own_stream;
+  return BLOK_OK;
+}
+
 extern "C" int blok_model_generate(blok_model_t *m, const uint32_t *prompt, int n_prompt, int max_new, uint32_t *out,
                                    int *n_out) {
   BLOK_REQUIRE(m && prompt && out && n_out, BLOK_ERR_ARG, "blok_model_generate: null pointer");
@@ -418,36 +427,39 @@ extern "C" int blok_model_generate(blok_model_t *m, const uint32_t *prompt, int 
     BLOK_REQUIRE(prompt[i] < (uint32_t)m->cfg.vocab, BLOK_ERR_ARG, "blok_model_generate: prompt token outside vocabulary");
   int rc = blok_model_reset(m);
   if (rc) return rc;
+  blok_stream_t stream;
+  if ((rc = generation_stream(m, &stream))) return rc;
   *n_out = 0;
   uint32_t next = prompt[0];
   if (m->cfg.prefill_chunk >= 1) {
     // the prompt in chunks: every layer's weights are read once per chunk instead of once per token
     BLOK_CUDA(cudaMemcpyAsync(m->prompt_ids, prompt, (size_t)n_prompt * 4, cudaMemcpyHostToDevice, nullptr));
-    if ((rc = blok_model_prefill(m, m->prompt_ids, n_prompt, m->next, nullptr))) return rc;
+    if ((rc = blok_model_prefill(m, m->prompt_ids, n_prompt, m->next, stream))) return rc;
   } else {
     // prompt replay, token by token; only the last step's sample is used (:886)
     for (int i = 0; i < n_prompt; ++i) {
       BLOK_CUDA(cudaMemcpyAsync(m->ids, prompt + i, 4, cudaMemcpyHostToDevice, nullptr));
-      if ((rc = blok_model_step(m, m->ids, 1, m->next, nullptr))) return rc;
+      if ((rc = blok_model_step(m, m->ids, 1, m->next, stream))) return rc;
     }
   }
   BLOK_CUDA(cudaMemcpy(&next, m->next, 4, cudaMemcpyDeviceToHost));
   for (int i = 0; i < max_new && next != m->cfg.eos_id; ++i) {  // :887-890
     out[(*n_out)++] = next;
     if (i + 1 < max_new) {
-      if ((rc = blok_model_step(m, m->next, 1, m->next, nullptr))) return rc;
+      if ((rc = blok_model_step(m, m->next, 1, m->next, stream))) return rc;
       BLOK_CUDA(cudaMemcpy(&next, m->next, 4, cudaMemcpyDeviceToHost));
     }
   }
   // a bounded device-side wait that gave up (or a position outside a cache) in any layer makes the tokens void
-  return blok_model_check(m, nullptr);
+  return blok_model_check(m, stream);
 }
 
 // The serving loop of blok_model_generate_many over an existing batcher (the caller destroys it).
 static int serve_requests(blok_model_t *m, blok_batcher_t *bt, const uint32_t *prompts, const int *prompt_offsets, int n_requests,
                           int max_new, uint32_t *out, int *n_out) {
   const blok_model_config &c = m->cfg;
-  int rc = BLOK_OK;
+  blok_stream_t stream;
+  int rc = generation_stream(m, &stream);
   for (int r = 0; r < n_requests && !rc; ++r) {
     int id = -1;
     rc = blok_batcher_submit(bt, prompt_offsets[r + 1] - prompt_offsets[r], max_new, &id);
@@ -466,7 +478,7 @@ static int serve_requests(blok_model_t *m, blok_batcher_t *bt, const uint32_t *p
     if (e) return e;
     if (finished) {
       slot_req[slot] = -1;
-      return blok_model_slot_release(m, slot, nullptr);
+      return blok_model_slot_release(m, slot, stream);
     }
     return BLOK_OK;
   };
@@ -481,7 +493,7 @@ static int serve_requests(blok_model_t *m, blok_batcher_t *bt, const uint32_t *p
     if (n_decode) {  // the running sequences step together; their ids come back for the EOS test, as at :882
       for (int b = 0; b < n_decode; ++b) ids[b] = last[decode_slots[b]];
       BLOK_CUDA(cudaMemcpyAsync(m->prompt_ids, ids.data(), (size_t)n_decode * 4, cudaMemcpyHostToDevice, nullptr));
-      if ((rc = blok_model_step_slots(m, decode_slots.data(), n_decode, m->prompt_ids, m->next, nullptr))) break;
+      if ((rc = blok_model_step_slots(m, decode_slots.data(), n_decode, m->prompt_ids, m->next, stream))) break;
       BLOK_CUDA(cudaMemcpy(sampled.data(), m->next, (size_t)n_decode * 4, cudaMemcpyDeviceToHost));
       for (int b = 0; b < n_decode && !rc; ++b) rc = take(decode_slots[b], sampled[b]);
       if (rc) break;
@@ -491,7 +503,7 @@ static int serve_requests(blok_model_t *m, blok_batcher_t *bt, const uint32_t *p
       const int n = prompt_offsets[r + 1] - prompt_offsets[r];
       slot_req[slot] = r;
       BLOK_CUDA(cudaMemcpyAsync(m->prompt_ids, prompts + prompt_offsets[r], (size_t)n * 4, cudaMemcpyHostToDevice, nullptr));
-      if ((rc = blok_model_prefill_slot(m, slot, m->prompt_ids, n, m->next, nullptr))) break;
+      if ((rc = blok_model_prefill_slot(m, slot, m->prompt_ids, n, m->next, stream))) break;
       uint32_t tok = 0;
       BLOK_CUDA(cudaMemcpy(&tok, m->next, 4, cudaMemcpyDeviceToHost));
       rc = take(slot, tok);
@@ -518,5 +530,5 @@ extern "C" int blok_model_generate_many(blok_model_t *m, const uint32_t *prompts
   if ((rc = blok_batcher_create(c.max_batch, c.kv_pages, c.kv_page_rows, c.max_ctx, &bt))) return rc;
   rc = serve_requests(m, bt, prompts, prompt_offsets, n_requests, max_new, out, n_out);
   blok_batcher_destroy(bt);
-  return rc ? rc : blok_model_check(m, nullptr);
+  return rc ? rc : blok_model_check(m, (blok_stream_t)m->own_stream);
 }

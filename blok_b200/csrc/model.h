@@ -63,6 +63,7 @@ struct blok_model {
   long long graph_launches[blok::kMaxBatch + 1] = {};  // kernels in each graph, added to the launch counter at every replay
   int steps_seen[blok::kMaxBatch + 1] = {};
   bool graphs_enabled = true;
+  cudaStream_t own_stream = nullptr;  // generation runs here: unlike the legacy default stream it can be captured
   // blok_model_trace_layers: fp32 [layer_runs, trace_rows, hidden]; layer_runs is set by the family's configure
   float *trace = nullptr;
   int trace_rows = 0, layer_runs = 0;

@@ -46,14 +46,22 @@ class Fields {
       }
     return out;
   }
-  Fields object(const char *name) { return Fields(rc_ ? nullptr : get(name), where_ + "." + name); }
+  // A field that is an object; after an error here its fields report nothing more.
+  Fields object(const char *name) {
+    const Json *v = get(name);
+    if (!rc_) return Fields(v, where_ + "." + name);
+    Fields none;
+    none.rc_ = rc_;
+    return none;
+  }
   void fail(const char *name, const char *what) { fail((std::string(name) + " " + what).c_str()); }
 
  private:
-  const Json *j_;
+  const Json *j_ = nullptr;
   std::string where_;
   int rc_ = BLOK_OK;
 
+  Fields() = default;
   const Json *get(const char *name) {
     if (rc_) return nullptr;
     const Json *v = j_->find(name);

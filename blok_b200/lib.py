@@ -682,6 +682,63 @@ class Batcher:
         return int(load().blok_batcher_emitted(self._handle, C.c_int(request)))
 
 
+def linear_attention(qkvg, heads, dim, vdim, decay, k_scale, silu, state, slot=0, first_pos=0, slot_of=None, pos=None):
+    """blok_linear_attention: qkvg [T, ld] bf16 or fp32, state fp32 [slots, heads, dim, vdim] updated -> o fp32 [T, heads * vdim]."""
+    T, ld = qkvg.shape
+    table = (C.c_float * (heads * 65))()
+    load().blok_linear_attention_decay((C.c_double * heads)(*decay), C.c_int(heads), table)
+    dev = torch.tensor(list(table), dtype=torch.float32, device=qkvg.device)
+    f = load().blok_linear_attention_scratch_bytes
+    f.restype = C.c_size_t
+    scratch = torch.empty(f(heads, dim, vdim, T), dtype=torch.uint8, device=qkvg.device)
+    o = torch.empty((T, heads * vdim), dtype=torch.float32, device=qkvg.device)
+    _check(load().blok_linear_attention(_ptr(qkvg), C.c_int(qkvg.dtype == torch.float32), C.c_int(ld), C.c_int(heads), C.c_int(dim), C.c_int(vdim),
+                                        _ptr(dev), C.c_float(k_scale), C.c_int(bool(silu)), _ptr(state, torch.float32, "state"), C.c_int(slot),
+                                        C.c_int(first_pos), C.c_int(T), _ptr(slot_of), _ptr(pos), _ptr(o), _ptr(scratch), _stream()))
+    return o
+
+
+def gated_norm(o, gate, heads, vdim, true_vdim, per_head, eps, sigmoid, w=None):
+    """blok_gated_norm: o fp32 [T, heads * vdim], gate bf16 or fp32 of the same shape."""
+    out = torch.empty_like(gate)
+    _check(load().blok_gated_norm(_ptr(o, torch.float32, "o"), _ptr(gate), C.c_int(gate.shape[1]), _ptr(w), C.c_int(heads), C.c_int(vdim),
+                                  C.c_int(true_vdim), C.c_int(bool(per_head)), C.c_float(eps), C.c_int(bool(sigmoid)), C.c_int(o.shape[0]),
+                                  _ptr(out), C.c_int(out.shape[1]), C.c_int(gate.dtype == torch.float32), _stream()))
+    return out
+
+
+def latent_attend(q, pool, table, slot_of, pos, rank, scale, max_ctx):
+    """blok_latent_attend: q [T, heads, rank + rot], pool [pages, page_rows, rank + rot], table int32 [slots, stride]."""
+    T, heads, row = q.shape
+    f = load().blok_latent_attend_workspace_bytes
+    f.restype = C.c_size_t
+    ws = torch.zeros(f(heads, row - rank, rank, T, C.c_long(max_ctx)), dtype=torch.uint8, device=q.device)
+    o = torch.empty((T, heads, rank), dtype=q.dtype, device=q.device)
+    _check(load().blok_latent_attend(_ptr(q), _ptr(pool), _ptr(table, torch.int32, "table"), C.c_int(table.shape[1]), C.c_int(pool.shape[1]),
+                                     _ptr(slot_of, torch.int32, "slot_of"), _ptr(pos, torch.int32, "pos"), C.c_int(heads), C.c_int(row - rank),
+                                     C.c_int(rank), C.c_float(scale), C.c_int(T), C.c_long(max_ctx), _ptr(o),
+                                     C.c_int(q.dtype == torch.float32), _ptr(ws), _stream()))
+    return o
+
+
+def latent_prompt(q, kv, k_rot, dim, vdim, scale):
+    """blok_latent_prompt: q [T, heads, dim + rot], kv [n, heads * (dim + vdim)], k_rot [n, rot] -> [T, heads * vdim]."""
+    T, heads, _ = q.shape
+    o = torch.empty((T, heads * vdim), dtype=torch.bfloat16, device=q.device)
+    _check(load().blok_latent_prompt(_ptr(q, torch.bfloat16, "q"), _ptr(kv, torch.bfloat16, "kv"), _ptr(k_rot, torch.bfloat16, "k_rot"),
+                                     C.c_int(heads), C.c_int(dim), C.c_int(k_rot.shape[1]), C.c_int(vdim), C.c_float(scale), C.c_int(T),
+                                     C.c_int(kv.shape[0]), _ptr(o), C.c_int(heads * vdim), _stream()))
+    return o
+
+
+def gemm_bf16(x, w, relu2=False, f32=True):
+    """blok_gemm_bf16: x [T, K], w [R, K] bf16 -> [T, R] fp32 (or bf16)."""
+    out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32 if f32 else torch.bfloat16, device=x.device)
+    _check(load().blok_gemm_bf16(_ptr(x, torch.bfloat16, "x"), _ptr(w, torch.bfloat16, "w"), C.c_int(x.shape[0]), C.c_int(w.shape[0]),
+                                 C.c_int(x.shape[1]), C.c_int(bool(relu2)), None if f32 else _ptr(out), _ptr(out) if f32 else None, _stream()))
+    return out
+
+
 class ModelConfig(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("layers", "first_dense", "hidden", "vocab", "dense_inter", "inter", "experts", "topk",
                                        "shared_inter")] + [("routed_scale", C.c_float)] + \

@@ -498,6 +498,44 @@ int blok_lm_head_argmax(const blok_bf16_t *w, const blok_bf16_t *n, int vocab, i
                         void *workspace, size_t workspace_bytes, blok_stream_t stream);
 
 /* ------------------------------------------------------------------------- */
+/* Mechanisms of the layer-stack models, one at a time                         */
+/* ------------------------------------------------------------------------- */
+
+/* Linear attention with a fixed decay per head: S_t = decay_h S_(t-1) + k_scale k_t v_t^T, o_t = S_t^T q_t, S fp32.
+ *   qkvg        bf16 (f32 = 0) or fp32 [T, ld]: q [heads * dim] | k [heads * dim] | v [heads * vdim] | anything
+ *   decay_table fp32 [heads, 65] of powers 0..64 on the device, made on the host by blok_linear_attention_decay
+ *   silu_qkv    q, k and v go through SiLU first
+ *   state       fp32 [slots, heads, dim, vdim], updated; o fp32 [T, heads * vdim]
+ * slot_of NULL: T consecutive tokens of the sequence in `slot`, the first at first_pos (0: the state starts at zero);
+ * scratch of blok_linear_attention_scratch_bytes for more than 8 bf16 tokens.  slot_of int32 [T] and pos int32 [T] (device):
+ * one token of each of T distinct sequences.  dim and vdim are multiples of 16, dim <= 256, ld of 8. */
+size_t blok_linear_attention_scratch_bytes(int heads, int dim, int vdim, int T);
+void blok_linear_attention_decay(const double *decay, int heads, float *table);
+int blok_linear_attention(const void *qkvg, int f32, int ld, int heads, int dim, int vdim, const float *decay_table,
+                          float k_scale, int silu_qkv, float *state, int slot, int first_pos, int T, const int *slot_of,
+                          const int *pos, float *o, void *scratch, blok_stream_t stream);
+/* out = o / rms(o) * w * gate(g), the mean square per head over true_vdim values (per_head) or over all heads; gate is SiLU
+ * or, with `sigmoid`, the logistic function.  o fp32 [T, heads * vdim], gate and out bf16 or fp32, w fp32 or NULL. */
+int blok_gated_norm(const float *o, const void *gate, int ld_gate, const float *w, int heads, int vdim, int true_vdim,
+                    int per_head, float eps, int sigmoid, int T, void *out, int ld_out, int f32, blok_stream_t stream);
+
+/* The cores of latent attention for any head count and sizes (blok_mla_attend is built for one).  Absorbed form: entry i
+ * attends to rows 0..pos[i] of the sequence in slot_of[i]; q [T, heads, rank + rot] and the pool's rows [rank + rot] are
+ * bf16 (fp32 with f32), o [T, heads, rank]; the softmax weights stay fp32.  rank and rot are multiples of 32.  The workspace
+ * must be zero before the first call and serve calls of one T and max_ctx only. */
+size_t blok_latent_attend_workspace_bytes(int heads, int rot, int rank, int T, long max_ctx);
+int blok_latent_attend(const void *q, const void *pool, const int *table, int table_stride, int page_rows,
+                       const int *slot_of, const int *pos, int heads, int rot, int rank, float scale, int T, long max_ctx,
+                       void *o, int f32, void *workspace, blok_stream_t stream);
+/* Prompt form: T queries at positions n - T .. n - 1 over n keys and values made from the latents: q [T, heads, dim + rot],
+ * kv [n, heads * dim | heads * vdim], k_rot [n, rot], o [T, ld_out].  dim + rot and vdim at most 256. */
+int blok_latent_prompt(const blok_bf16_t *q, const blok_bf16_t *kv, const blok_bf16_t *k_rot, int heads, int dim, int rot,
+                       int vdim, float scale, int T, int n, blok_bf16_t *o, int ld_out, blok_stream_t stream);
+/* out[t, r] = act(sum_k x[t, k] w[r, k]) on tcgen05 with TMA-fed tiles; act: none, or the square of ReLU. */
+int blok_gemm_bf16(const blok_bf16_t *x, const blok_bf16_t *w, int T, int R, int K, int relu2, blok_bf16_t *out_bf16,
+                   float *out_f32, blok_stream_t stream);
+
+/* ------------------------------------------------------------------------- */
 /* A11/A12  whole model: decode step and greedy generation (config 4)          */
 /* ------------------------------------------------------------------------- */
 

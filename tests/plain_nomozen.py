@@ -16,7 +16,7 @@ def bf16_round(a):
     """float32 array rounded to the nearest bfloat16 value (ties to even), returned as float32."""
     u = np.ascontiguousarray(a, np.float32).view(np.uint32)
     r = ((u + 0x7FFF + ((u >> 16) & 1)) & np.uint32(0xFFFF0000)).astype(np.uint32)
-    return r.view(np.float32)
+    return r.view(np.float32).reshape(np.shape(a))
 
 
 def read_safetensors(path):
@@ -242,9 +242,9 @@ def random_model(cfg, seed, gain=1.0):
             t[p + "mlp.table"] = np.stack([rng.permutation(E)[:k] for _ in range(V)]).astype(np.int32)
             hcs.append("hc2")
         for hc in hcs:
-            vec(p + hc + ".in", S, 1.0 / S, 0.3)
+            vec(p + hc + ".in", S, 1.0 / S, 0.3 / S)
             vec(p + hc + ".out", S, 1.0, 0.3)
-            t[p + hc + ".mix"] = bf16_round((0.8 * np.eye(S) + 0.2 * rng.normal(size=(S, S))).astype(np.float32))
+            t[p + hc + ".mix"] = bf16_round((0.7 * np.eye(S) + 0.3 / S * rng.normal(size=(S, S))).astype(np.float32))
     norm("final.norm")
     mat("head", V, W, 2.0)
     return t
