@@ -313,6 +313,126 @@ def ep_measure(T, rank, world, device, comm, steps, warmup, experts=384):
     return rec, launches
 
 
+NOMOZEN_SIZES = {
+    # width, experts per layer, experts per token, expert size, linear-attention heads; attention as config 3 (64 heads)
+    "small": dict(width=2048, experts=128, top=8, ff=1024, heads=16),
+    "large": dict(width=7168, experts=128, top=8, ff=2048, heads=56),
+}
+
+
+def nomozen_config(width, experts, top, ff, heads, vocab=32768):
+    """A four-layer Nomozen model of a real model's layer sizes: retention, two latent-attention layers, lightning."""
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    linear = {"heads": heads, "dim": 128, "vdim": 128, "decay": [1 - 2.0 ** -(5 + 5 * h / heads) for h in range(heads)]}
+    latent = {"heads": 64, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 1536, "scale": 192 ** -0.5,
+              "rot": {"base": 50000.0, "dims": 64}}
+    layers = [{"type": "retention", "mixer": linear}, {"type": "latent_attention", "mixer": latent},
+              {"type": "latent_attention", "mixer": latent}, {"type": "lightning", "mixer": linear}]
+    return {"architecture": "Nomozen", "width": width, "vocab": vocab, "streams": 4, "norm": {"eps": 1e-5},
+            "layers": [dict(l, mlp=mlp) for l in layers]}
+
+
+def nomozen_bytes(c, batch, ctx):
+    """Algorithmic bytes of one decode step: every weight the step touches once, states and latent rows once, the streams."""
+    W, total = c["width"], 0
+    for l in c["layers"]:
+        m, f = l["mixer"], l["mlp"]
+        if l["type"] == "latent_attention":
+            row = m["kv_rank"] + m["rot_dim"]
+            w = m["q_rank"] * W + row * W + m["heads"] * (m["dim"] + m["rot_dim"]) * m["q_rank"] + m["heads"] * m["dim"] * m["kv_rank"] + \
+                m["heads"] * m["vdim"] * m["kv_rank"] + W * m["heads"] * m["vdim"]
+            total += 2 * w + batch * ctx * row * 2
+        else:
+            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            total += 2 * W * (2 * hd + 2 * hv + hv) + batch * m["heads"] * m["dim"] * m["vdim"] * 8
+        e, k = f["router"]["experts"], f["router"]["top"]
+        touched = e * (1 - (1 - k / e) ** batch)     # expected distinct experts of a batch
+        total += int(touched * 2 * W * f["expert"]["ff"] * 2) + 2 * batch * 2 * c["streams"] * W * 4
+    return total + c["vocab"] * W * 2
+
+
+def nomozen_workload(a, device, steps, warmup):
+    """Decode and prompt throughput of a Nomozen model beside the library's Kimi model at equal sizes (four layers each, the
+    same width, attention, expert count and size; Kimi's experts are INT4 and have three matrices), one GPU.  --impl-only
+    runs one of the two (profiler launch lists)."""
+    import torch
+    from blok_b200 import lib
+    size = NOMOZEN_SIZES[a.size]
+    B, ctx, P = a.batch, a.ctx, a.prompt
+    cfg = nomozen_config(**size)
+    vocab = cfg["vocab"]
+    max_ctx = max(ctx, P) + steps + max(warmup, 3) + 16
+    pages = B * ((max_ctx + 63) // 64) + ((P + 63) // 64)
+    peak, peak_kind = measured_peak()
+    kinds = {"nomozen": lambda: lib.Model.open_synthetic(cfg, seed=4, max_batch=B + 1, max_ctx=max_ctx, prefill_chunk=min(2048, max(P, ctx)), kv_pages=pages),
+             "kimi": lambda: lib.Model(seed=4, layers=4, first_dense=0, hidden=size["width"], vocab=vocab, inter=size["ff"], experts=size["experts"],
+                                       topk=size["top"], shared_inter=size["ff"], max_batch=B + 1, max_ctx=max_ctx, prefill_chunk=64,
+                                       kv_page_rows=64, kv_pages=pages)}
+    sampler = ClockSampler(device.index or 0)
+    sampler.start()
+    out, launches = {}, 0
+    for kind in ([a.impl_only] if a.impl_only else ["nomozen", "kimi"]):
+        model = kinds[kind]()
+        side = torch.cuda.Stream()
+        torch.cuda.synchronize()
+        with torch.cuda.stream(side):
+            prompts = [torch.randint(0, vocab, (max(P, ctx),), device=device, dtype=torch.int32) for _ in range(4)]
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            rec = {}
+            if P:
+                def prompt(i):
+                    model.prefill_slot(B, prompts[i % 4][:P])
+                    model.release_slot(B)
+                n = max(2, steps // 4)
+                for i in range(2 if a.impl_only else 3):
+                    prompt(i)
+                side.synchronize()
+                l0 = lib.kernel_launch_count()
+                e0.record()
+                for i in range(n):
+                    prompt(i)
+                e1.record()
+                side.synchronize()
+                launches += lib.kernel_launch_count() - l0
+                rec["prefill_ms"] = e0.elapsed_time(e1) / n
+                rec["prefill_tok_per_s"] = P / (rec["prefill_ms"] * 1e-3)
+            if ctx:
+                for b in range(B):
+                    model.prefill_slot(b, prompts[b % 4][:ctx])
+                slots = list(range(B))
+                ids = torch.randint(0, vocab, (B,), device=device, dtype=torch.int32)
+                for _ in range(max(warmup, 3)):
+                    ids = model.step_slots(slots, ids)
+                side.synchronize()
+                l0 = lib.kernel_launch_count()
+                e0.record()
+                for _ in range(steps):
+                    ids = model.step_slots(slots, ids)
+                e1.record()
+                side.synchronize()
+                launches += lib.kernel_launch_count() - l0
+                rec["decode_ms"] = e0.elapsed_time(e1) / steps
+                rec["decode_tok_per_s"] = B / (rec["decode_ms"] * 1e-3)
+                if kind == "nomozen":
+                    alg = nomozen_bytes(cfg, B, ctx)
+                    rec["decode_roofline"] = {"bound": "hbm", "bytes": alg, "achieved": alg / (rec["decode_ms"] * 1e-3) / 1e9, "peak": peak,
+                                              "unit": "GB/s", "frac": alg / (rec["decode_ms"] * 1e-3) / 1e9 / peak, "peak_kind": peak_kind}
+            model.check()
+        model.close()
+        out[kind] = rec
+    clocks = sampler.stop()
+    main = out.get("nomozen", out.get("kimi"))
+    print(json.dumps({
+        "metric": "decode tok/s, 4-layer Nomozen model (batch %d, ctx %d)" % (B, ctx), "value": main.get("decode_tok_per_s"), "unit": "tok/s",
+        "n_gpus": 1, "steps": steps, "warmup": warmup, "ms_per_step": main.get("decode_ms"), "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "Nomozen beside Kimi's model at equal size (%s: %s), four layers each, %d-token prompts, paged caches" %
+                               (a.size, json.dumps(size), P),
+                   "l2": "a step reads more weights than the L2 holds; prompts rotated"},
+        **out, "gpu_launches": int(launches), "clocks": clocks}))
+    return 0
+
+
 def other_workload(a, rank, world, device, steps, warmup):
     """Configs 2 and 3 through the same timing rules (CUDA events, barrier both sides, max over ranks)."""
     import torch
@@ -586,9 +706,14 @@ def main():
     ap.add_argument("--experts", type=int, default=384,
                     help="routed experts per layer; below 384 the run is a reduced case for profiler captures, "
                          "not the benchmark configuration, and the line says so")
-    ap.add_argument("--workload", default="decode", choices=["decode", "expert", "batched64", "batched2048", "mla4096", "mla32768", "model", "model61", "prefill512", "gemv"],
+    ap.add_argument("--size", default="large", choices=sorted(NOMOZEN_SIZES), help="layer sizes of the `nomozen` workload")
+    ap.add_argument("--ctx", type=int, default=4096, help="cached tokens per sequence of the `nomozen` workload (0: no decoding)")
+    ap.add_argument("--prompt", type=int, default=1024, help="prompt length of the `nomozen` workload (0: no prompts)")
+    ap.add_argument("--impl-only", default=None, choices=["nomozen", "kimi"], help="one side of the `nomozen` workload")
+    ap.add_argument("--workload", default="decode", choices=["decode", "expert", "batched64", "batched2048", "mla4096", "mla32768", "model", "model61", "prefill512", "gemv", "nomozen"],
                     help="decode = config 1 (the default, the headline metric); batched* = config 2 (expert parallel "
-                         "when --gpus > 1); mla* = config 3 (attention block, batch 8)")
+                         "when --gpus > 1); mla* = config 3 (attention block, batch 8); nomozen = a Nomozen model beside "
+                         "Kimi's at equal size, one GPU (--size, --batch, --ctx, --prompt)")
     a = ap.parse_args()
 
     import torch
@@ -625,6 +750,8 @@ def main():
     if world > 1:
         dist.init_process_group("nccl", device_id=device)
     lib.load()
+    if a.workload == "nomozen":
+        return nomozen_workload(a, device, steps if a.steps is not None else 20, warmup if a.warmup is not None else 5)
     if a.workload != "decode":
         return other_workload(a, rank, world, device, steps if a.steps is not None else 20, warmup if a.warmup is not None else 5)
 

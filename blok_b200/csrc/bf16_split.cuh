@@ -8,11 +8,17 @@ namespace blok {
 
 constexpr int kSplitParts = 3;
 
+// Both values rounded to nearest even, a in the low half, in one instruction.
+__device__ __forceinline__ uint32_t pack_pair(float a, float b) {
+  uint32_t r;
+  asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r) : "f"(b), "f"(a));
+  return r;
+}
 // Parts of the pair (a, b) as packed bf16 pairs, a in the low half.
 __device__ __forceinline__ void split_pair(float a, float b, uint32_t (&parts)[kSplitParts]) {
 #pragma unroll
   for (int p = 0; p < kSplitParts; ++p) {
-    const uint32_t v = pack_bf16x2(a, b);
+    const uint32_t v = pack_pair(a, b);
     parts[p] = v;
     a -= bf16lo(v);
     b -= bf16hi(v);

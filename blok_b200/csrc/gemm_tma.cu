@@ -33,7 +33,7 @@ __device__ unsigned g_gemm_tma_error = 0;
 struct GtArgs {
   void *out;
   const int *tile_expert, *tile_start, *tile_count, *num_tiles;
-  int T, R, K, ldo;
+  int T, R, K, ldo, act_cols;
 };
 
 template <int ACT>
@@ -42,6 +42,7 @@ __device__ __forceinline__ float gt_act(float v) {
     v = fmaxf(v, 0.f);
     return v * v;
   }
+  if (ACT == GEMM_ACT_SILU) return v / (1.0f + expf(-v));
   return v;
 }
 
@@ -139,8 +140,8 @@ __global__ void __launch_bounds__(kGtThreads)
           for (int j = 0; j < 32; j += 4) {
             const int col = n0 + c0 + j;
             if (col < a.R) {  // R is a multiple of 4
-              const float f0 = gt_act<ACT>(__uint_as_float(v[j])), f1 = gt_act<ACT>(__uint_as_float(v[j + 1]));
-              const float f2 = gt_act<ACT>(__uint_as_float(v[j + 2])), f3 = gt_act<ACT>(__uint_as_float(v[j + 3]));
+              float f0 = __uint_as_float(v[j]), f1 = __uint_as_float(v[j + 1]), f2 = __uint_as_float(v[j + 2]), f3 = __uint_as_float(v[j + 3]);
+              if (ACT != GEMM_ACT_SILU || col < a.act_cols) f0 = gt_act<ACT>(f0), f1 = gt_act<ACT>(f1), f2 = gt_act<ACT>(f2), f3 = gt_act<ACT>(f3);
               if (F32) *reinterpret_cast<float4 *>(static_cast<float *>(a.out) + o + col) = make_float4(f0, f1, f2, f3);
               else *reinterpret_cast<uint2 *>(static_cast<uint16_t *>(a.out) + o + col) = make_uint2(pack_bf16x2(f0, f1), pack_bf16x2(f2, f3));
             }
@@ -184,7 +185,7 @@ int gemm_operand_map(const void *base, long rows, int cols, long pitch, int box,
 
 template <int BN, int ACT, bool F32>
 static int gt_launch(const GemmTma &g, dim3 grid, cudaStream_t stream) {
-  const GtArgs a = {g.out, g.tile_expert, g.tile_start, g.tile_count, g.num_tiles, g.T, g.R, g.K, g.ldo};
+  const GtArgs a = {g.out, g.tile_expert, g.tile_start, g.tile_count, g.num_tiles, g.T, g.R, g.K, g.ldo, g.act_cols};
   BLOK_CUDA(cudaFuncSetAttribute(gemm_tma_kernel<BN, ACT, F32>, cudaFuncAttributeMaxDynamicSharedMemorySize, GtCfg<BN>::kSmem));
   gemm_tma_kernel<BN, ACT, F32><<<grid, kGtThreads, GtCfg<BN>::kSmem, stream>>>(*g.x, BN == 128 ? *g.w128 : *g.w256, a);
   return launch_status("gemm_tma_kernel");
@@ -197,6 +198,10 @@ int launch_gemm_tma(const GemmTma &g, cudaStream_t stream) {
   const long wide = (long)((g.R + 255) / 256) * (g.tile_start ? (g.T + kGtTileRows - 1) / kGtTileRows : tiles);
   const bool use256 = g.w256 && wide >= sm_count();
   const dim3 grid((g.R + (use256 ? 255 : 127)) / (use256 ? 256 : 128), tiles);
+  if (g.act == GEMM_ACT_SILU) {
+    BLOK_REQUIRE(!g.out_f32 && g.act_cols % 4 == 0, BLOK_ERR_SHAPE, "gemm: SiLU on %d columns of an fp32 output", g.act_cols);
+    return use256 ? gt_launch<256, GEMM_ACT_SILU, false>(g, grid, stream) : gt_launch<128, GEMM_ACT_SILU, false>(g, grid, stream);
+  }
 #define BLOK_GT(BN)                                                                                   \
   return g.act == GEMM_ACT_RELU2 ? (g.out_f32 ? gt_launch<BN, GEMM_ACT_RELU2, true>(g, grid, stream)   \
                                               : gt_launch<BN, GEMM_ACT_RELU2, false>(g, grid, stream)) \

@@ -7,7 +7,7 @@
 
 namespace blok {
 
-enum { GEMM_ACT_NONE = 0, GEMM_ACT_RELU2 = 1 };
+enum { GEMM_ACT_NONE = 0, GEMM_ACT_RELU2 = 1, GEMM_ACT_SILU = 2 };
 constexpr int kGtTileRows = 128;  // rows of x per tile
 
 // A matrix operand: bf16 [rows, cols], rows `pitch` elements apart (pitch a multiple of 8, base 16-byte aligned).
@@ -23,6 +23,7 @@ struct GemmTma {
   bool out_f32 = false;
   int ldo = 0;
   int act = GEMM_ACT_NONE;
+  int act_cols = 0;                            // GEMM_ACT_SILU: the first so many columns (a multiple of 4) only; bf16 output
   // Grouped form: tile i covers rows [tile_start[i], + tile_count[i]) of x (at most kGtTileRows) and weight rows
   // [tile_expert[i] * R, + R); at most max_tiles tiles, *num_tiles of them valid.  NULL: consecutive tiles of one matrix.
   const int *tile_expert = nullptr, *tile_start = nullptr, *tile_count = nullptr, *num_tiles = nullptr;

@@ -4,12 +4,15 @@
 // Two forms, both causal.  Absorbed (decode, short portions): queries multiplied by W_UK^T score against the cached rows
 // themselves and the latents are averaged, one pass over the cache, the context split over CTAs (mla_merge.cuh adds the
 // parts).  Prompt form (long portions): per-head keys and values are made from the cached latents by one product and a
-// tile kernel walks them, which needs 3 to 4 times fewer multiply-adds per query and key.
+// tile kernel walks them, which needs 3 to 4 times fewer multiply-adds per query and key (latent_prompt_tc.cu on tcgen05 for
+// sizes in multiples of 64, the mma.sync kernel here for the others).
 //
 // Scores, softmax and its weights are fp32; the weights enter the second product in three bf16 parts (bf16_split.cuh).
 // Positions become angles in double precision.  (The cores of mla_attend.cu and mla_attend_tc.cu are built for 64 heads of
 // one size and round the weights to bf16.)
 #include <algorithm>
+#include <cstdlib>
+#include <cstring>
 
 #include "bf16_split.cuh"
 #include "mla_merge.cuh"
@@ -30,15 +33,15 @@ __device__ __forceinline__ void lt_store(Act *p, float v) {
 __device__ __forceinline__ size_t lt_row(const StackRows &r, int slot, int pos) {
   return (size_t)r.table[(size_t)slot * r.table_stride + pos / r.page_rows] * r.page_rows + pos % r.page_rows;
 }
-// Sine and cosine of pos * base^(-2i / dims), reduced to one turn in double.
-__device__ __forceinline__ void lt_angle(int pos, int i, int dims, double log2_base, float *s, float *c) {
-  const double turns = (double)pos * exp2(-2.0 * i / dims * log2_base) * 0.15915494309189533577;
+// Sine and cosine at position pos of a pair that makes `rate` turns per position, reduced to one turn in double.
+__device__ __forceinline__ void lt_angle(int pos, double rate, float *s, float *c) {
+  const double turns = (double)pos * rate;
   sincosf((float)((turns - rint(turns)) * 6.28318530717958647693), s, c);
 }
 
 // ---- norms of the latents, rotation of the shared key part, cache append; one CTA per token ----
 template <typename Act>
-__global__ void __launch_bounds__(256) latent_append_kernel(const LatentShape s, double log2_base, const float *__restrict__ ckr, const float *__restrict__ q_norm,
+__global__ void __launch_bounds__(256) latent_append_kernel(const LatentShape s, const float *__restrict__ ckr, const float *__restrict__ q_norm,
                                                             const float *__restrict__ kv_norm, const StackRows r, Act *__restrict__ cq,
                                                             Act *__restrict__ pool) {
   __shared__ float s_red[2][8];
@@ -65,7 +68,7 @@ __global__ void __launch_bounds__(256) latent_append_kernel(const LatentShape s,
     float u = k[2 * i], v = k[2 * i + 1];
     if (2 * i < s.rot_dims) {
       float sn, cs;
-      lt_angle(pos, i, s.rot_dims, log2_base, &sn, &cs);
+      lt_angle(pos, s.turns[i], &sn, &cs);
       const float a = u * cs - v * sn;
       v = v * cs + u * sn;
       u = a;
@@ -77,20 +80,19 @@ __global__ void __launch_bounds__(256) latent_append_kernel(const LatentShape s,
 
 int launch_latent_append(const LatentShape &s, const float *ckr, const float *q_norm, const float *kv_norm, const StackRows &r, int T, void *cq,
                          void *pool, bool f32, cudaStream_t stream) {
-  const double lb = log2(s.rot_base);
-  if (f32) latent_append_kernel<float><<<T, 256, 0, stream>>>(s, lb, ckr, q_norm, kv_norm, r, static_cast<float *>(cq), static_cast<float *>(pool));
-  else latent_append_kernel<uint16_t><<<T, 256, 0, stream>>>(s, lb, ckr, q_norm, kv_norm, r, static_cast<uint16_t *>(cq), static_cast<uint16_t *>(pool));
+  if (f32) latent_append_kernel<float><<<T, 256, 0, stream>>>(s, ckr, q_norm, kv_norm, r, static_cast<float *>(cq), static_cast<float *>(pool));
+  else latent_append_kernel<uint16_t><<<T, 256, 0, stream>>>(s, ckr, q_norm, kv_norm, r, static_cast<uint16_t *>(cq), static_cast<uint16_t *>(pool));
   return launch_status("latent_append_kernel");
 }
 
 template <typename Act>
-__global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentShape s, double log2_base, const Act *q, const StackRows r, int T, Act *dst,
+__global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentShape s, const Act *q, const StackRows r, int T, Act *dst,
                                                             int dst_head, int dst_off) {
   extern __shared__ float2 s_sc[];  // sine and cosine of every pair at this token's position
   const int t = blockIdx.x, pos = r.pos[t], half = s.rot / 2;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn = 0.f, cs = 1.f;
-    if (2 * i < s.rot_dims) lt_angle(pos, i, s.rot_dims, log2_base, &sn, &cs);
+    if (2 * i < s.rot_dims) lt_angle(pos, s.turns[i], &sn, &cs);
     s_sc[i] = make_float2(sn, cs);
   }
   __syncthreads();
@@ -107,11 +109,10 @@ __global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentShape s,
 
 int launch_latent_rotate(const LatentShape &s, const void *q, const StackRows &r, int T, void *dst, int dst_head, int dst_off, bool f32,
                          cudaStream_t stream) {
-  const double lb = log2(s.rot_base);
   const dim3 grid(T, T >= 64 ? 1 : std::max(1, s.heads * (s.rot / 2) / 512));
   const size_t smem = (size_t)(s.rot / 2) * sizeof(float2);
-  if (f32) latent_rotate_kernel<float><<<grid, 256, smem, stream>>>(s, lb, static_cast<const float *>(q), r, T, static_cast<float *>(dst), dst_head, dst_off);
-  else latent_rotate_kernel<uint16_t><<<grid, 256, smem, stream>>>(s, lb, static_cast<const uint16_t *>(q), r, T, static_cast<uint16_t *>(dst), dst_head, dst_off);
+  if (f32) latent_rotate_kernel<float><<<grid, 256, smem, stream>>>(s, static_cast<const float *>(q), r, T, static_cast<float *>(dst), dst_head, dst_off);
+  else latent_rotate_kernel<uint16_t><<<grid, 256, smem, stream>>>(s, static_cast<const uint16_t *>(q), r, T, static_cast<uint16_t *>(dst), dst_head, dst_off);
   return launch_status("latent_rotate_kernel");
 }
 
@@ -207,13 +208,15 @@ __global__ void __launch_bounds__(kLaThreads, 1)
     const int h = u / units, c = u - h * units;  // heads past the last repeat it; their results are not stored
     cp_async16(qs + h * pitch + c * 16, q_abs + ((size_t)b * s.heads + h0 + min(h, nh - 1)) * row + c * 8);
   }
+  // a row of the tile belongs to four neighbouring threads: one look into the page table per thread and tile
+  constexpr int kRowThreads = kLaThreads / kLaTile;
+  const int lk = tid / kRowThreads, lc = tid % kRowThreads;
   auto load_tile = [&](int tile, int buf) {
-    for (int u = tid; u < kLaTile * units; u += kLaThreads) {
-      const int k = u / units, c = u - k * units;
-      const int j = min(tile * kLaTile + k, n - 1);  // rows past the end repeat the last; they take no weight
-      const size_t at = (size_t)table[j / r.page_rows] * r.page_rows + j % r.page_rows;
-      cp_async16(ks + (uint32_t)(buf * kLaTile + k) * pitch + c * 16, pool + at * row + c * 8);
-    }
+    const int j = min(tile * kLaTile + lk, n - 1);  // rows past the end repeat the last; they take no weight
+    const uint16_t *src = pool + ((size_t)table[j / r.page_rows] * r.page_rows + j % r.page_rows) * row;
+    const uint32_t dst = ks + (uint32_t)(buf * kLaTile + lk) * pitch;
+#pragma unroll 6
+    for (int c = lc; c < units; c += kRowThreads) cp_async16(dst + c * 16, src + c * 8);
   };
   load_tile(ts, 0);
   asm volatile("cp.async.commit_group;" ::: "memory");
@@ -343,6 +346,20 @@ __global__ void __launch_bounds__(kLaThreads, 1)
   }
 }
 
+int launch_mla_attend_tc_fine(const uint16_t *q, const uint16_t *pool, long pool_rows, const int *block_table, const int *slot_of, int table_stride,
+                              int page_rows, const int *pos, int B, int heads, int splits, float scale, float *part_o, float *part_ml,
+                              cudaStream_t stream);
+
+// The tcgen05 core (mla_attend_tc.cu) is built for rows of 512 + 64 values and takes heads 64 at a time; fewer than 24 are
+// better off with the kernel above.  BLOK_MLA_ATTEND_IMPL=mma (read at every call) switches it off.
+static bool la_fine(const LatentShape &s, int page_rows) {
+  const char *impl = getenv("BLOK_MLA_ATTEND_IMPL");
+  return s.scale > 0.f && s.rank == 512 && s.rot == 64 && s.heads >= 24 && page_rows % 64 == 0 && !(impl && strcmp(impl, "mma") == 0);
+}
+static int la_fine_splits(const LatentShape &s, int T, long max_ctx) {
+  const int groups = (s.heads + 63) / 64;
+  return (int)std::max(1l, std::min((max_ctx + 63) / 64, (long)(sm_count() / (groups * T))));
+}
 static bool la_tensor(const LatentShape &s) { return s.rank <= kLaMaxRank && la_smem_bytes(s, s.heads > 16 ? 2 : 1) <= 227 * 1024; }
 static int la_splits(const LatentShape &s, int T, long max_ctx) {
   const int groups = (s.heads + (s.heads > 16 ? 31 : 15)) / (s.heads > 16 ? 32 : 16);
@@ -352,7 +369,7 @@ static int la_splits(const LatentShape &s, int T, long max_ctx) {
 
 size_t latent_attend_max_parts(const LatentShape &s, int T, long max_ctx) {
   size_t worst = 0;
-  for (int t = 1; t <= T; ++t) worst = std::max(worst, (size_t)t * la_splits(s, t, max_ctx));
+  for (int t = 1; t <= T; ++t) worst = std::max(worst, (size_t)t * std::max(la_splits(s, t, max_ctx), la_fine_splits(s, t, max_ctx)));
   return worst;
 }
 
@@ -382,14 +399,18 @@ int launch_latent_attend(const LatentShape &s, const void *q_abs, const void *po
     }
     return launch_status("latent_attend_simple_kernel");
   }
-  const int splits = la_splits(s, T, max_ctx);
+  const bool fine = la_fine(s, r.page_rows);
+  const int splits = fine ? la_fine_splits(s, T, max_ctx) : la_splits(s, T, max_ctx);
   const uint16_t *q = static_cast<const uint16_t *>(q_abs), *p = static_cast<const uint16_t *>(pool);
   int rc;
 #define BLOK_LA(MT)                                                                        \
   rc = s.rank <= 128   ? la_launch<MT, 2>(s, q, p, r, T, splits, part_o, part_ml, stream)  \
        : s.rank <= 256 ? la_launch<MT, 4>(s, q, p, r, T, splits, part_o, part_ml, stream)  \
                        : la_launch<MT, 8>(s, q, p, r, T, splits, part_o, part_ml, stream)
-  if (s.heads > 16) BLOK_LA(2);
+  if (fine)  // a tile never leaves its page: the pool needs no tighter bound than the coordinate range
+    rc = launch_mla_attend_tc_fine(q, p, (1l << 31) - 64, r.table, r.slot_of, r.table_stride, r.page_rows, r.pos, T, s.heads, splits, s.scale, part_o,
+                                   part_ml, stream);
+  else if (s.heads > 16) BLOK_LA(2);
   else BLOK_LA(1);
 #undef BLOK_LA
   if (rc) return rc;
@@ -563,6 +584,10 @@ __global__ void __launch_bounds__(kLpThreads, 1)
   }
 }
 
+bool latent_prompt_tc_supports(const LatentShape &s);
+int launch_latent_prompt_tc(const LatentShape &s, const uint16_t *q, const uint16_t *kv, const uint16_t *kr_all, int T, int n, uint16_t *o, int ldo,
+                            cudaStream_t stream);
+
 bool latent_prompt_supports(const LatentShape &s) { return s.head() <= 256 && s.vdim <= 256; }
 
 template <int DQ, int DV>
@@ -577,6 +602,8 @@ static int lp_launch(const LatentShape &s, const uint16_t *q, const uint16_t *kv
 int launch_latent_prompt(const LatentShape &s, const uint16_t *q, const uint16_t *kv, const uint16_t *kr_all, int T, int n, uint16_t *o, int ldo,
                          cudaStream_t stream) {
   BLOK_REQUIRE(latent_prompt_supports(s) && n >= T && T >= 1, BLOK_ERR_SHAPE, "latent attention: heads of %d / %d", s.head(), s.vdim);
+  const char *impl = getenv("BLOK_MLA_ATTEND_IMPL");
+  if (latent_prompt_tc_supports(s) && !(impl && strcmp(impl, "mma") == 0)) return launch_latent_prompt_tc(s, q, kv, kr_all, T, n, o, ldo, stream);
   if (s.head() <= 96 && s.vdim <= 64) return lp_launch<96, 64>(s, q, kv, kr_all, T, n, o, ldo, stream);
   if (s.head() <= 128 && s.vdim <= 128) return lp_launch<128, 128>(s, q, kv, kr_all, T, n, o, ldo, stream);
   if (s.head() <= 192 && s.vdim <= 128) return lp_launch<192, 128>(s, q, kv, kr_all, T, n, o, ldo, stream);

@@ -1,0 +1,296 @@
+// The prompt form of latent attention (latent_attn.cu) on tcgen05: causal attention of T queries over n per-head keys and
+// values, for a query-key size of 128 to 256 and a value size of 64 or 128, in multiples of 64.
+//
+// A CTA owns 128 queries of one head and walks the keys in tiles of 64:
+//   S [queries x 64]   = Q K^T    both operands in shared memory (TMA, 128-byte swizzle), accumulator in tensor memory, two
+//                                 buffers
+//   P = exp2(S * scale * log2 e - m)   one query per thread: no exchange between threads for its maximum and sum
+//   O [queries x vdim] += P V     P in tensor memory as the A operand, in three bf16 parts (bf16_split.cuh); V is read from
+//                                 its rows as they are (MN-major B operand)
+// The scores of tile n + 1 are computed under the softmax of tile n.  The running maximum is kept lazily: a row's reference
+// moves, and its 64 or 128 accumulators are rescaled, only when a tile's maximum exceeds it by more than 40 natural units.
+//
+// Warps: 0..3 softmax (a warp reaches its own 32 lanes of tensor memory), 4: copies, 5: MMA.  Every wait is bounded; a CTA that
+// gives up records it, waits for its copies in flight, releases its tensor memory and returns.  No copy is multicast.
+#include <mutex>
+
+#include "bf16_split.cuh"
+#include "gemm_tma.h"
+#include "stack_kernels.h"
+#include "tc_pipe.cuh"
+
+namespace blok {
+
+constexpr int kPtRows = 128, kPtKeys = 64, kPtStages = 3, kPtThreads = 192;
+constexpr int kPtQChunk = kPtRows * 128, kPtKChunk = kPtKeys * 128;  // bytes of a 64-column chunk
+constexpr int kPtMaxQ = 4;                                           // chunks of a query
+constexpr int kPtColS = 0, kPtColP = 128, kPtColO = 384;             // tensor memory: S 2 x 64, P 2 x 3 x 32 (of 4 x 64), O
+constexpr int kPtTmemCols = 512;
+constexpr float kPtLazy = 57.7f;  // 40 natural units in the log2 domain
+
+__device__ unsigned g_latent_prompt_error = 0;
+
+__device__ __forceinline__ float pt_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+struct PtArgs {
+  uint16_t *out;
+  int T, n, ldo, heads, dim, rot, vdim;
+  float scale_log2;
+};
+
+__global__ void __launch_bounds__(kPtThreads, 1)
+    latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mkv, const __grid_constant__ CUtensorMap mkr,
+                            const PtArgs a) {
+  extern __shared__ unsigned char smem_raw[];
+  __shared__ __align__(8) unsigned long long s_bar[2 * kPtStages + 9];
+  __shared__ uint32_t s_tmem;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, q0 = (gridDim.x - 1 - blockIdx.x) * kPtRows;  // the longest rows of tiles start first
+  const int first = a.n - a.T, nq = min(kPtRows, a.T - q0);
+  const int nt = (first + q0 + nq + kPtKeys - 1) / kPtKeys;
+  const int qc = (a.dim + a.rot) / 64, dc = a.dim / 64, vc = a.vdim / 64;
+  const uint32_t sQ = ((uint32_t)__cvta_generic_to_shared(smem_raw) + 1023u) & ~1023u;
+  const uint32_t stage_bytes = (uint32_t)(qc + vc) * kPtKChunk, sT = sQ + (uint32_t)qc * kPtQChunk;
+  const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&s_bar[0]);
+  const uint32_t full = bar, empty = bar + 8 * kPtStages, qfull = bar + 16 * kPtStages, sfull = qfull + 8, sfree = qfull + 24, pfull = qfull + 40,
+                 pdone = qfull + 56;
+  if (tid == 0) {
+    for (int s = 0; s < kPtStages; ++s) {
+      tp_mbar_init(full + 8 * s, 1);
+      tp_mbar_init(empty + 8 * s, 1);
+    }
+    tp_mbar_init(qfull, 1);
+    for (int b = 0; b < 2; ++b) {
+      tp_mbar_init(sfull + 8 * b, 1);
+      tp_mbar_init(sfree + 8 * b, 4);
+      tp_mbar_init(pfull + 8 * b, 4);
+      tp_mbar_init(pdone + 8 * b, 1);
+    }
+    tp_mbar_init_fence();
+  }
+  if (warp == 0) tp_tmem_alloc((uint32_t)__cvta_generic_to_shared(&s_tmem), kPtTmemCols);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = s_tmem;
+  bool failed = false;
+
+  if (warp == 4) {
+    if (lane == 0) {
+      tp_expect_tx(qfull, (uint32_t)qc * kPtQChunk);
+      for (int c = 0; c < qc; ++c) tp_load_2d(sQ + c * kPtQChunk, &mq, h * (a.dim + a.rot) + 64 * c, q0, qfull);
+      int issued = 0;
+      for (int n = 0; n < nt; ++n) {
+        const int s = n % kPtStages;
+        if (n >= kPtStages && !tp_wait(empty + 8 * s, (uint32_t)((n / kPtStages - 1) & 1))) {
+          failed = true;
+          break;
+        }
+        const uint32_t dst = sT + (uint32_t)s * stage_bytes, f = full + 8 * s;
+        tp_expect_tx(f, stage_bytes);
+        for (int c = 0; c < dc; ++c) tp_load_2d(dst + c * kPtKChunk, &mkv, h * a.dim + 64 * c, n * kPtKeys, f);
+        for (int c = dc; c < qc; ++c) tp_load_2d(dst + c * kPtKChunk, &mkr, 64 * (c - dc), n * kPtKeys, f);
+        for (int c = 0; c < vc; ++c) tp_load_2d(dst + (qc + c) * kPtKChunk, &mkv, a.heads * a.dim + h * a.vdim + 64 * c, n * kPtKeys, f);
+        issued = n + 1;
+      }
+      // no copy may be in flight when the CTA leaves
+      tp_wait(qfull, 0);
+      for (int n = max(0, issued - kPtStages); n < issued; ++n) tp_wait(full + 8 * (n % kPtStages), (uint32_t)((n / kPtStages) & 1));
+    }
+  } else if (warp == 5) {
+    if (lane == 0) {
+      const uint32_t idesc_s = tp_idesc_bf16(kPtKeys), idesc_pv = tp_idesc_bf16(a.vdim) | (1u << 16);  // V: MN-major B operand
+      auto issue_s = [&](int n) {
+        const uint32_t k = sT + (uint32_t)(n % kPtStages) * stage_bytes;
+        for (int c = 0; c < qc; ++c) {
+          const uint64_t qd = tp_desc_k_sw128(sQ + c * kPtQChunk), kd = tp_desc_k_sw128(k + c * kPtKChunk);
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            tp_mma(tmem + kPtColS + 64 * (n & 1), qd + (uint64_t)(2 * j), kd + (uint64_t)(2 * j), idesc_s, (c | j) ? 1u : 0u);
+        }
+        tp_commit(sfull + 8 * (n & 1));
+      };
+      failed = !tp_wait(qfull, 0) || !tp_wait(full, 0);
+      if (!failed) {
+        tc_fence_after();
+        issue_s(0);
+      }
+      for (int n = 0; n < nt && !failed; ++n) {
+        const int b = n & 1;
+        if (n + 1 < nt) {
+          const int m = n + 1;
+          if (!tp_wait(full + 8 * (m % kPtStages), (uint32_t)((m / kPtStages) & 1)) ||
+              (m >= 2 && !tp_wait(sfree + 8 * (m & 1), (uint32_t)(((m >> 1) - 1) & 1)))) {
+            failed = true;
+            break;
+          }
+          tc_fence_after();
+          issue_s(m);
+        }
+        if (!tp_wait(pfull + 8 * b, (uint32_t)((n >> 1) & 1))) {
+          failed = true;
+          break;
+        }
+        tc_fence_after();
+        const uint64_t vd = tp_desc_mn_sw128(sT + (uint32_t)(n % kPtStages) * stage_bytes + qc * kPtKChunk, kPtKChunk);
+#pragma unroll
+        for (int p = 0; p < kSplitParts; ++p)
+#pragma unroll
+          for (int j = 0; j < kPtKeys / 16; ++j)
+            tp_mma_ts(tmem + kPtColO, tmem + kPtColP + 128 * b + 32 * p + 8 * j, vd + (uint64_t)(j * (2048 >> 4)), idesc_pv, (n | p | j) ? 1u : 0u);
+        tp_commit(empty + 8 * (n % kPtStages));
+        tp_commit(pdone + 8 * b);
+      }
+    }
+  } else {
+    const uint32_t lanes = (uint32_t)(32 * warp) << 16;
+    const int pos = first + q0 + tid;        // this thread's query
+    const int warp_first = first + q0 + 32 * warp;
+    float m_ref = 0.f, l = 0.f;
+    for (int n = 0; n < nt; ++n) {
+      const int b = n & 1;
+      failed = !tp_wait(sfull + 8 * b, (uint32_t)((n >> 1) & 1));
+      if (__any_sync(0xffffffffu, failed)) {
+        failed = true;
+        break;
+      }
+      tc_fence_after();
+      uint32_t r[64];
+      tmem_ld64(tmem + lanes + kPtColS + 64 * b, r);
+      tmem_wait_ld();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) tp_arrive(sfree + 8 * b);
+      if (n * kPtKeys + kPtKeys - 1 > warp_first) {  // keys behind a query take no weight
+#pragma unroll
+        for (int j = 0; j < 64; ++j)
+          if (n * kPtKeys + j > pos) r[j] = 0xff800000u;
+      }
+      float x0 = -INFINITY, x1 = -INFINITY, x2 = -INFINITY, x3 = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < 64; j += 4) {
+        x0 = fmaxf(x0, __uint_as_float(r[j]));
+        x1 = fmaxf(x1, __uint_as_float(r[j + 1]));
+        x2 = fmaxf(x2, __uint_as_float(r[j + 2]));
+        x3 = fmaxf(x3, __uint_as_float(r[j + 3]));
+      }
+      const float mx = fmaxf(fmaxf(x0, x1), fmaxf(x2, x3)) * a.scale_log2;  // the scale is positive
+      float alpha = 1.f;
+      bool need = false;
+      if (n == 0) {
+        m_ref = mx;  // position 0 is in this tile and every query sees it
+      } else if (mx > m_ref + kPtLazy) {
+        alpha = pt_ex2(m_ref - mx);
+        m_ref = mx;
+        need = true;
+      }
+      const float nm = -m_ref;
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < 64; j += 2) {
+        const float p0 = pt_ex2(fmaf(__uint_as_float(r[j]), a.scale_log2, nm)), p1 = pt_ex2(fmaf(__uint_as_float(r[j + 1]), a.scale_log2, nm));
+        s0 += p0;
+        s1 += p1;
+        r[j] = __float_as_uint(p0);
+        r[j + 1] = __float_as_uint(p1);
+      }
+      l = l * alpha + (s0 + s1);
+      if (n >= 2) failed = !tp_wait(pdone + 8 * b, (uint32_t)(((n >> 1) - 1) & 1));  // the products of tile n - 2 have read this buffer
+      if (__any_sync(0xffffffffu, need) && n >= 1) failed = failed || !tp_wait(pdone + 8 * (b ^ 1), (uint32_t)(((n - 1) >> 1) & 1));
+      if (__any_sync(0xffffffffu, failed)) {
+        failed = true;
+        break;
+      }
+      tc_fence_after();
+      if (__any_sync(0xffffffffu, need)) {
+#pragma unroll 1
+        for (int c = 0; c < vc; ++c) {
+          uint32_t o[64];
+          tmem_ld64(tmem + lanes + kPtColO + 64 * c, o);
+          tmem_wait_ld();
+#pragma unroll
+          for (int j = 0; j < 64; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * alpha);
+          tmem_st64(tmem + lanes + kPtColO + 64 * c, o);
+        }
+      }
+#pragma unroll
+      for (int p = 0; p < kSplitParts; ++p) {
+        uint32_t w[32];
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          const float u = __uint_as_float(r[2 * j]), v = __uint_as_float(r[2 * j + 1]);
+          w[j] = pack_pair(u, v);
+          r[2 * j] = __float_as_uint(u - bf16lo(w[j]));
+          r[2 * j + 1] = __float_as_uint(v - bf16hi(w[j]));
+        }
+        tmem_st32(tmem + lanes + kPtColP + 128 * b + 32 * p, w);
+      }
+      tmem_wait_st();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) tp_arrive(pfull + 8 * b);
+    }
+    if (!failed) failed = !tp_wait(pdone + 8 * ((nt - 1) & 1), (uint32_t)(((nt - 1) >> 1) & 1));
+    failed = __any_sync(0xffffffffu, failed);
+    if (!failed) {
+      tc_fence_after();
+      const float inv = 1.0f / l;
+      uint16_t *o = a.out + (size_t)(q0 + tid) * a.ldo + (size_t)h * a.vdim;
+#pragma unroll 1
+      for (int c = 0; c < 2 * vc; ++c) {
+        uint32_t v[32];
+        tmem_ld32(tmem + lanes + kPtColO + 32 * c, v);
+        tmem_wait_ld();
+        if (tid < nq) {
+#pragma unroll
+          for (int j = 0; j < 32; j += 8) {
+            uint32_t w[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) w[k] = pack_bf16x2(__uint_as_float(v[j + 2 * k]) * inv, __uint_as_float(v[j + 2 * k + 1]) * inv);
+            *reinterpret_cast<uint4 *>(o + 32 * c + j) = make_uint4(w[0], w[1], w[2], w[3]);
+          }
+        }
+      }
+    }
+  }
+  if (failed) atomicExch(&g_latent_prompt_error, 1u);
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) tp_tmem_free(tmem, kPtTmemCols);
+}
+
+bool latent_prompt_tc_supports(const LatentShape &s) {
+  return s.scale > 0.f && s.dim % 64 == 0 && s.rot % 64 == 0 && s.head() <= 64 * kPtMaxQ && (s.vdim == 64 || s.vdim == 128);
+}
+
+int launch_latent_prompt_tc(const LatentShape &s, const uint16_t *q, const uint16_t *kv, const uint16_t *kr_all, int T, int n, uint16_t *o, int ldo,
+                            cudaStream_t stream) {
+  BLOK_REQUIRE(ldo % 8 == 0, BLOK_ERR_SHAPE, "latent attention: rows of %d outputs", ldo);
+  CUtensorMap mq, mkv, mkr;
+  const int qw = s.heads * s.head(), kw = s.heads * (s.dim + s.vdim);
+  int rc;
+  // rows past the last query and key read as zeros
+  if ((rc = gemm_operand_map(q, T, qw, qw, kPtRows, &mq)) || (rc = gemm_operand_map(kv, n, kw, kw, kPtKeys, &mkv)) ||
+      (rc = gemm_operand_map(kr_all, n, s.rot, s.rot, kPtKeys, &mkr)))
+    return rc;
+  const PtArgs a = {o, T, n, ldo, s.heads, s.dim, s.rot, s.vdim, s.scale * 1.4426950408889634f};
+  const int qc = s.head() / 64, vc = s.vdim / 64;
+  const int smem = qc * kPtQChunk + kPtStages * (qc + vc) * kPtKChunk + 1024;
+  BLOK_CUDA(cudaFuncSetAttribute(latent_prompt_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  latent_prompt_tc_kernel<<<dim3((T + kPtRows - 1) / kPtRows, s.heads), kPtThreads, smem, stream>>>(mq, mkv, mkr, a);
+  return launch_status("latent_prompt_tc_kernel");
+}
+
+// *out becomes non-zero if a CTA has given up on a barrier since the last call (the flag is cleared).
+int latent_prompt_take_error(unsigned *out) {
+  unsigned zero = 0;
+  BLOK_CUDA(cudaMemcpyFromSymbol(out, g_latent_prompt_error, sizeof(unsigned)));
+  if (*out) BLOK_CUDA(cudaMemcpyToSymbol(g_latent_prompt_error, &zero, sizeof(unsigned)));
+  return BLOK_OK;
+}
+
+}  // namespace blok

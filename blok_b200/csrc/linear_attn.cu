@@ -103,26 +103,33 @@ __global__ void __launch_bounds__(256) linear_recurrent_kernel(const LaArgs a) {
 }
 
 // ---- chunked form ----
-constexpr int kLcThreads = 128;
+constexpr int kLcThreads = 256;
+constexpr int kLcAhead = 4;  // loads in flight per thread while a tile is staged
 constexpr int kLcCols = 64;  // columns of v per CTA
 constexpr int kLcVPitch = kLcCols * 2 + 16;
 
+__device__ __forceinline__ uint4 lc_silu8(uint4 v) {
+  uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) w[j] = pack_bf16x2(la_silu(bf16lo(w[j])), la_silu(bf16hi(w[j])));
+  return make_uint4(w[0], w[1], w[2], w[3]);
+}
+
 // `n` rows of `cols` bf16 (a multiple of 8) from p (row pitch ld elements) into a tile; rows past n are zero.
 __device__ __forceinline__ void lc_stage(unsigned char *dst, int pitch, const uint16_t *p, int ld, int n, int cols, bool silu) {
-  const int per = cols / 8;
-  for (int u = threadIdx.x; u < kLinChunk * per; u += kLcThreads) {
-    const int r = u / per, c = u - r * per;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < n) {
-      v = *reinterpret_cast<const uint4 *>(p + (size_t)r * ld + c * 8);
-      if (silu) {
-        uint32_t w[4] = {v.x, v.y, v.z, v.w};
+  const int per = cols / 8, total = kLinChunk * per;
+  for (int u0 = threadIdx.x; u0 < total; u0 += kLcAhead * kLcThreads) {
+    uint4 v[kLcAhead];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) w[j] = pack_bf16x2(la_silu(bf16lo(w[j])), la_silu(bf16hi(w[j])));
-        v = make_uint4(w[0], w[1], w[2], w[3]);
-      }
+    for (int q = 0; q < kLcAhead; ++q) {
+      const int u = u0 + q * kLcThreads, r = u / per, c = u - r * per;
+      v[q] = u < total && r < n ? *reinterpret_cast<const uint4 *>(p + (size_t)r * ld + c * 8) : make_uint4(0, 0, 0, 0);
     }
-    *reinterpret_cast<uint4 *>(dst + (size_t)r * pitch + c * 16) = v;
+#pragma unroll
+    for (int q = 0; q < kLcAhead; ++q) {
+      const int u = u0 + q * kLcThreads, r = u / per, c = u - r * per;
+      if (u < total) *reinterpret_cast<uint4 *>(dst + (size_t)r * pitch + c * 16) = silu ? lc_silu8(v[q]) : v[q];
+    }
   }
 }
 
@@ -137,30 +144,35 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_state_kernel(const La
   const float *pw = a.decay_pow + h * (kLinChunk + 1);
   const uint16_t *rows = static_cast<const uint16_t *>(a.qkvg) + (size_t)c * kLinChunk * a.ld;
   const uint16_t *k = rows + (size_t)a.heads * a.dim + (size_t)h * a.dim;
-  for (int u = threadIdx.x; u < kLinChunk * (a.dim / 8); u += kLcThreads) {  // the decayed keys in three parts
-    const int r = u / (a.dim / 8), col = (u - r * (a.dim / 8)) * 8;
-    uint32_t part[4][kSplitParts] = {};
-    if (r < n) {
-      const uint4 x = *reinterpret_cast<const uint4 *>(k + (size_t)r * a.ld + col);
-      const uint32_t w[4] = {x.x, x.y, x.z, x.w};
-      const float wt = a.k_scale * pw[n - 1 - r];
+  const int per = a.dim / 8, total = kLinChunk * per;
+  for (int u0 = threadIdx.x; u0 < total; u0 += kLcAhead * kLcThreads) {  // the decayed keys in three parts
+    uint4 x[kLcAhead];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        float lo = bf16lo(w[j]), hi = bf16hi(w[j]);
-        if (a.silu) lo = round_bf16(la_silu(lo)), hi = round_bf16(la_silu(hi));
-        split_pair(lo * wt, hi * wt, part[j]);
-      }
+    for (int q = 0; q < kLcAhead; ++q) {
+      const int u = u0 + q * kLcThreads, r = u / per;
+      x[q] = u < total && r < n ? *reinterpret_cast<const uint4 *>(k + (size_t)r * a.ld + (u - r * per) * 8) : make_uint4(0, 0, 0, 0);
     }
 #pragma unroll
-    for (int p = 0; p < kSplitParts; ++p)
-      *reinterpret_cast<uint4 *>(smem + (size_t)(p * kLinChunk + r) * kp + col * 2) = make_uint4(part[0][p], part[1][p], part[2][p], part[3][p]);
+    for (int q = 0; q < kLcAhead; ++q) {
+      const int u = u0 + q * kLcThreads, r = u / per, col = (u - r * per) * 8;
+      if (u >= total) break;
+      if (a.silu) x[q] = lc_silu8(x[q]);
+      const float wt = r < n ? a.k_scale * pw[n - 1 - r] : 0.f;
+      const uint32_t w[4] = {x[q].x, x[q].y, x[q].z, x[q].w};
+      uint32_t part[4][kSplitParts];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) split_pair(bf16lo(w[j]) * wt, bf16hi(w[j]) * wt, part[j]);
+#pragma unroll
+      for (int p = 0; p < kSplitParts; ++p)
+        *reinterpret_cast<uint4 *>(smem + (size_t)(p * kLinChunk + r) * kp + col * 2) = make_uint4(part[0][p], part[1][p], part[2][p], part[3][p]);
+    }
   }
   lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)a.heads * a.dim + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
   __syncthreads();
   const uint32_t ks = (uint32_t)__cvta_generic_to_shared(smem), vs = (uint32_t)__cvta_generic_to_shared(Vs);
   float *out = a.chunk_state + (((size_t)c * a.heads + h) * a.dim) * a.vdim + v0;
   const int g = lane >> 2, t = lane & 3;
-  for (int m0 = warp * 16; m0 < a.dim; m0 += 64) {
+  for (int m0 = warp * 16; m0 < a.dim; m0 += 16 * (kLcThreads / 32)) {
     float acc[kLcCols / 8][4] = {};
 #pragma unroll
     for (int k0 = 0; k0 < kLinChunk; k0 += 16) {
@@ -217,8 +229,8 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LaArgs a) {
   *st = s;
 }
 
-// grid = (chunks, heads, columns / 64); a warp owns 16 tokens of the chunk.
-__global__ void __launch_bounds__(kLcThreads) linear_chunk_out_kernel(const LaArgs a) {
+// grid = (chunks, heads, columns / 64); a warp owns 16 tokens of the chunk and half of the columns.
+__global__ void __launch_bounds__(kLcThreads, 2) linear_chunk_out_kernel(const LaArgs a) {
   extern __shared__ __align__(16) unsigned char smem[];
   __shared__ float s_pw[kLinChunk + 1];
   const int c = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * kLcCols;
@@ -233,22 +245,33 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_out_kernel(const LaAr
   lc_stage(Ks, kp, rows + hd + (size_t)h * a.dim, a.ld, n, a.dim, a.silu);
   lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)hd + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
   const float *S = a.chunk_state + (((size_t)c * a.heads + h) * a.dim) * a.vdim + v0;
-  for (int u = threadIdx.x; u < a.dim * (vc / 4); u += kLcThreads) {  // the state in three parts
-    const int r = u / (vc / 4), col = (u - r * (vc / 4)) * 4;
-    const float4 x = *reinterpret_cast<const float4 *>(S + (size_t)r * a.vdim + col);
-    uint32_t p0[kSplitParts], p1[kSplitParts];
-    split_pair(x.x, x.y, p0);
-    split_pair(x.z, x.w, p1);
+  const int per = vc / 4, total = a.dim * per;
+  for (int u0 = threadIdx.x; u0 < total; u0 += kLcAhead * kLcThreads) {  // the state in three parts
+    float4 x[kLcAhead];
 #pragma unroll
-    for (int p = 0; p < kSplitParts; ++p)
-      *reinterpret_cast<uint2 *>(Ss + (size_t)(p * a.dim + r) * kLcVPitch + col * 2) = make_uint2(p0[p], p1[p]);
+    for (int q = 0; q < kLcAhead; ++q) {
+      const int u = u0 + q * kLcThreads, r = u / per;
+      x[q] = u < total ? *reinterpret_cast<const float4 *>(S + (size_t)r * a.vdim + (u - r * per) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int q = 0; q < kLcAhead; ++q) {
+      const int u = u0 + q * kLcThreads, r = u / per, col = (u - r * per) * 4;
+      if (u >= total) break;
+      uint32_t p0[kSplitParts], p1[kSplitParts];
+      split_pair(x[q].x, x[q].y, p0);
+      split_pair(x[q].z, x[q].w, p1);
+#pragma unroll
+      for (int p = 0; p < kSplitParts; ++p)
+        *reinterpret_cast<uint2 *>(Ss + (size_t)(p * a.dim + r) * kLcVPitch + col * 2) = make_uint2(p0[p], p1[p]);
+    }
   }
   __syncthreads();
-  const int m0 = warp * 16;
-  if (m0 >= n) return;  // no barrier follows
+  const int m0 = (warp & 3) * 16, c0 = (warp >> 2) * (kLcCols / 2);
+  if (m0 >= n || c0 >= vc) return;  // no barrier follows
+  constexpr int kTiles = kLcCols / 16;  // the warp's column tiles of 8
   const uint32_t qs = (uint32_t)__cvta_generic_to_shared(smem), ks = (uint32_t)__cvta_generic_to_shared(Ks);
   const uint32_t vs = (uint32_t)__cvta_generic_to_shared(Vs), ss = (uint32_t)__cvta_generic_to_shared(Ss);
-  float sc[kLinChunk / 8][4] = {}, acc[kLcCols / 8][4] = {};
+  float sc[kLinChunk / 8][4] = {}, acc[kTiles][4] = {};
   for (int k0 = 0; k0 < a.dim; k0 += 16) {
     uint32_t q0, q1, q2, q3;
     ldsm4(frag_a(qs, m0, k0, kp, lane), q0, q1, q2, q3);
@@ -262,12 +285,12 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_out_kernel(const LaAr
       }
     }
 #pragma unroll
-    for (int nt = 0; nt < kLcCols / 8; nt += 2) {
-      if (nt * 8 < vc) {
+    for (int nt = 0; nt < kTiles; nt += 2) {
+      if (c0 + nt * 8 < vc) {
 #pragma unroll
         for (int p = 0; p < kSplitParts; ++p) {
           uint32_t b0, b1, b2, b3;
-          ldsm4_t(frag_b_t(ss + p * a.dim * kLcVPitch, nt * 8, k0, kLcVPitch, lane), b0, b1, b2, b3);
+          ldsm4_t(frag_b_t(ss + p * a.dim * kLcVPitch, c0 + nt * 8, k0, kLcVPitch, lane), b0, b1, b2, b3);
           mma_bf16_16816(acc[nt], q0, q1, q2, q3, b0, b1);
           mma_bf16_16816(acc[nt + 1], q0, q1, q2, q3, b2, b3);
         }
@@ -277,7 +300,7 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_out_kernel(const LaAr
   // the state's share decays by one step more than the token's place in the chunk
   const float d_lo = s_pw[m0 + g + 1], d_hi = s_pw[m0 + g + 9];
 #pragma unroll
-  for (int nt = 0; nt < kLcCols / 8; ++nt) {
+  for (int nt = 0; nt < kTiles; ++nt) {
     acc[nt][0] *= d_lo;
     acc[nt][1] *= d_lo;
     acc[nt][2] *= d_hi;
@@ -298,10 +321,10 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_out_kernel(const LaAr
         split_pair(w2, w3, fa[2 * half + 1]);
       }
 #pragma unroll
-      for (int nt = 0; nt < kLcCols / 8; nt += 2) {
-        if (nt * 8 < vc) {
+      for (int nt = 0; nt < kTiles; nt += 2) {
+        if (c0 + nt * 8 < vc) {
           uint32_t b0, b1, b2, b3;
-          ldsm4_t(frag_b_t(vs, nt * 8, kk * 16, kLcVPitch, lane), b0, b1, b2, b3);
+          ldsm4_t(frag_b_t(vs, c0 + nt * 8, kk * 16, kLcVPitch, lane), b0, b1, b2, b3);
 #pragma unroll
           for (int p = 0; p < kSplitParts; ++p) {
             mma_bf16_16816(acc[nt], fa[0][p], fa[1][p], fa[2][p], fa[3][p], b0, b1);
@@ -314,9 +337,9 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_out_kernel(const LaAr
   const int hv = a.heads * a.vdim;
   float *o = a.o + (size_t)c * kLinChunk * hv + (size_t)h * a.vdim + v0;
 #pragma unroll
-  for (int nt = 0; nt < kLcCols / 8; ++nt) {
-    if (nt * 8 < vc) {
-      const int col = nt * 8 + 2 * t;
+  for (int nt = 0; nt < kTiles; ++nt) {
+    if (c0 + nt * 8 < vc) {
+      const int col = c0 + nt * 8 + 2 * t;
       if (i_lo < n) *reinterpret_cast<float2 *>(o + (size_t)i_lo * hv + col) = make_float2(acc[nt][0], acc[nt][1]);
       if (i_hi < n) *reinterpret_cast<float2 *>(o + (size_t)i_hi * hv + col) = make_float2(acc[nt][2], acc[nt][3]);
     }
@@ -331,25 +354,73 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNorm a) {
   const float *o = a.o + (size_t)blockIdx.x * n;
   const Act *g = static_cast<const Act *>(a.g) + (size_t)blockIdx.x * a.ldg;
   Act *out = static_cast<Act *>(a.out) + (size_t)blockIdx.x * a.ldo;
-  auto write = [&](int i, float scale) {
-    const float z = la_load(g + i), e = 1.0f / (1.0f + expf(-z));
-    const float v = o[i] * scale * (a.w ? a.w[i] : 1.f) * (a.gate == GATE_SILU ? z * e : e);
-    if constexpr (sizeof(Act) == 2) out[i] = f32_to_bf16_bits(v);
-    else out[i] = v;
+  auto gates4 = [&](int i) {  // columns i .. i + 3 of the gate
+    if constexpr (sizeof(Act) == 2) {
+      const uint2 v = *reinterpret_cast<const uint2 *>(g + i);
+      return make_float4(bf16lo(v.x), bf16hi(v.x), bf16lo(v.y), bf16hi(v.y));
+    } else {
+      return *reinterpret_cast<const float4 *>(g + i);
+    }
   };
+  auto write4 = [&](int i, float4 v, float4 gate, float scale) {
+    const float x[4] = {v.x, v.y, v.z, v.w}, zs[4] = {gate.x, gate.y, gate.z, gate.w};
+    float r[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float z = zs[j], e = 1.0f / (1.0f + expf(-z));
+      r[j] = x[j] * scale * (a.w ? a.w[i + j] : 1.f) * (a.gate == GATE_SILU ? z * e : e);
+    }
+    if constexpr (sizeof(Act) == 2) *reinterpret_cast<uint2 *>(out + i) = make_uint2(pack_bf16x2(r[0], r[1]), pack_bf16x2(r[2], r[3]));
+    else *reinterpret_cast<float4 *>(out + i) = make_float4(r[0], r[1], r[2], r[3]);
+  };
+  auto sq = [](float4 v, float s) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s)))); };
+  constexpr int kKeep = 8;  // a thread's values stay in registers between the sum and the scaling; longer rows are read again
+  float4 keep[kKeep];
   if (a.per_head) {
-    for (int h = blockIdx.y * 8 + warp; h < a.heads; h += 8 * gridDim.y) {
+    const int step = 8 * gridDim.y;
+    int h = blockIdx.y * 8 + warp;
+    if (a.vdim <= 128) {  // a lane holds four columns of a head: four heads in flight per warp
+      const int i = lane * 4;
+      const bool in = i < a.vdim;
+      for (; h < a.heads; h += 4 * step) {
+        float4 v[4], z[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const bool ok = in && h + q * step < a.heads;
+          v[q] = ok ? *reinterpret_cast<const float4 *>(o + (h + q * step) * a.vdim + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+          z[q] = ok ? gates4((h + q * step) * a.vdim + i) : v[q];
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const float scale = 1.0f / sqrtf(warp_sum(sq(v[q], 0.f)) / (float)a.true_vdim + a.eps);
+          if (in && h + q * step < a.heads) write4((h + q * step) * a.vdim + i, v[q], z[q], scale);
+        }
+      }
+    }
+    for (; h < a.heads; h += step) {
       float s = 0.f;
-      for (int i = lane; i < a.vdim; i += 32) s = fmaf(o[h * a.vdim + i], o[h * a.vdim + i], s);
+#pragma unroll
+      for (int k = 0; k < kKeep; ++k) {
+        const int i = (lane + 32 * k) * 4;
+        if (i < a.vdim) s = sq(keep[k] = *reinterpret_cast<const float4 *>(o + h * a.vdim + i), s);
+      }
+      for (int i = (lane + 32 * kKeep) * 4; i < a.vdim; i += 128) s = sq(*reinterpret_cast<const float4 *>(o + h * a.vdim + i), s);
       const float scale = 1.0f / sqrtf(warp_sum(s) / (float)a.true_vdim + a.eps);
-      for (int i = lane; i < a.vdim; i += 32) write(h * a.vdim + i, scale);
+#pragma unroll
+      for (int k = 0; k < kKeep; ++k) {
+        const int i = (lane + 32 * k) * 4;
+        if (i < a.vdim) write4(h * a.vdim + i, keep[k], gates4(h * a.vdim + i), scale);
+      }
+      for (int i = (lane + 32 * kKeep) * 4; i < a.vdim; i += 128) write4(h * a.vdim + i, *reinterpret_cast<const float4 *>(o + h * a.vdim + i), gates4(h * a.vdim + i), scale);
     }
   } else {
     float s = 0.f;
-    for (int i = tid * 4; i < n; i += 1024) {
-      const float4 v = *reinterpret_cast<const float4 *>(o + i);
-      s = fmaf(v.x, v.x, s), s = fmaf(v.y, v.y, s), s = fmaf(v.z, v.z, s), s = fmaf(v.w, v.w, s);
+#pragma unroll
+    for (int k = 0; k < kKeep; ++k) {
+      const int i = (tid + 256 * k) * 4;
+      if (i < n) s = sq(keep[k] = *reinterpret_cast<const float4 *>(o + i), s);
     }
+    for (int i = (tid + 256 * kKeep) * 4; i < n; i += 1024) s = sq(*reinterpret_cast<const float4 *>(o + i), s);
     s = warp_sum(s);
     if (lane == 0) s_red[warp] = s;
     __syncthreads();
@@ -357,8 +428,14 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNorm a) {
 #pragma unroll
     for (int w = 0; w < 8; ++w) s += s_red[w];
     const float scale = 1.0f / sqrtf(s / (float)(a.heads * a.true_vdim) + a.eps);
-    const int per = (n + gridDim.y - 1) / gridDim.y, end = min(n, (int)(blockIdx.y + 1) * per);
-    for (int i = blockIdx.y * per + tid; i < end; i += 256) write(i, scale);
+    // several CTAs of one token: CTA y writes every gridDim.y-th group of 1,024 columns
+#pragma unroll
+    for (int k = 0; k < kKeep; ++k) {
+      const int i = (tid + 256 * k) * 4;
+      if (k % gridDim.y == blockIdx.y && i < n) write4(i, keep[k], gates4(i), scale);
+    }
+    for (int k = kKeep, i = (tid + 256 * kKeep) * 4; i < n; ++k, i += 1024)
+      if (k % gridDim.y == blockIdx.y) write4(i, *reinterpret_cast<const float4 *>(o + i), gates4(i), scale);
   }
   if (blockIdx.y == 0)
     for (int i = n + tid; i < a.ldo; i += 256) out[i] = Act(0);

@@ -74,7 +74,26 @@ __global__ void argmax_f32_kernel(const float *__restrict__ logits, int vocab, i
   const float *row = logits + (size_t)blockIdx.x * pitch;
   float best = -INFINITY;
   int bi = 0x7fffffff;
-  for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
+  // four loads of four logits in flight per thread, in ascending order
+  const int units = pitch % 4 == 0 ? vocab / 4 : 0;
+  const float4 *row4 = reinterpret_cast<const float4 *>(row);
+  for (int u0 = threadIdx.x; u0 < units; u0 += 4 * blockDim.x) {
+    float4 q[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int u = u0 + k * blockDim.x;
+      q[k] = u < units ? row4[u] : make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i0 = (u0 + k * blockDim.x) * 4;
+      if (q[k].x > best) best = q[k].x, bi = i0;
+      if (q[k].y > best) best = q[k].y, bi = i0 + 1;
+      if (q[k].z > best) best = q[k].z, bi = i0 + 2;
+      if (q[k].w > best) best = q[k].w, bi = i0 + 3;
+    }
+  }
+  for (int i = units * 4 + threadIdx.x; i < vocab; i += blockDim.x) {
     const float v = row[i];
     if (v > best) best = v, bi = i;
   }

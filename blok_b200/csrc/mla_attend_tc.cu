@@ -22,6 +22,11 @@
 // 40 (natural units); then all four consumer warps rescale O^T in tensor memory.  exp(s - m) stays far inside fp32 and
 // bf16 range meanwhile, and the merge over the splits needs a consistent (m, sum, O) only.
 //
+// FINE: the weights enter the second product as two bf16 parts, high and low (17 bits of each weight; the sum of the weights
+// is fp32), for models whose attention weights are fp32.  The low part needs no shared memory of its own: a tile's chunk of
+// rope columns is read by the score product only, so once the tile's scores have been taken the low parts go there, and
+// the tile's release frees both.  seq_len then holds positions (the token itself included).  Any number of heads in groups of 64 (blockIdx.z).
+//
 // Warps: 0..3 consumers (the M = 64 accumulator S keeps head rows 16 w .. 16 w + 15 in lanes 0..15 of warp w's quarter of
 // tensor memory; all four own the 128 lanes of O^T), 4: the TMA producer, 5: one lane issues the MMAs.  Every mbarrier
 // wait is bounded; on a timeout the CTA records an error, still releases its tensor memory and returns.
@@ -156,12 +161,12 @@ size_t mla_attend_tc_smem_bytes() { return kTaSmemBytes; }
 
 // grid = (splits, B); arguments as mla_attend_kernel, plus the tensor map of the cache ([rows, 576] bf16, boxes of
 // 64 rows x 64 columns, 128-byte swizzle).  PAGED: page_rows is a multiple of the 64-token tile.
-template <bool PAGED>
+template <bool PAGED, bool FINE>
 __global__ void __launch_bounds__(kTaThreads, 1)
     mla_attend_tc_kernel(const __grid_constant__ CUtensorMap tmap, const uint16_t *__restrict__ q, const uint16_t *__restrict__ cache,
                          long ctx_stride, const int *__restrict__ seq_len, float scale, float *__restrict__ part_o,
                          float *__restrict__ part_ml, const int *__restrict__ block_table, const int *__restrict__ slot_of,
-                         int table_stride, int page_rows, long long *__restrict__ trace) {
+                         int table_stride, int page_rows, long long *__restrict__ trace, int heads) {
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(8) unsigned long long s_bar[11];
   __shared__ uint32_t s_tmem;
@@ -169,13 +174,14 @@ __global__ void __launch_bounds__(kTaThreads, 1)
   __shared__ int s_need[2][4];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int split = blockIdx.x, splits = gridDim.x, b = blockIdx.y;
-  const int seq = seq_len[b];
+  const int seq = FINE ? min(seq_len[b] + 1, table_stride * page_rows) : seq_len[b];
   const int ntiles = (seq + kTaTile - 1) / kTaTile;
   const int per = (ntiles + splits - 1) / splits;
   const int ts = split * per, te = min(ntiles, ts + per);
-  float *my_ml = part_ml + ((size_t)b * splits + split) * kTaHeads * 2;
+  const int h0 = blockIdx.z * kTaHeads, nh = min(kTaHeads, heads - h0);  // this CTA's heads
+  float *my_ml = part_ml + (((size_t)b * splits + split) * heads + h0) * 2;
   if (ts >= te) {  // nothing to do for this split: mark it empty for the merge
-    if (tid < kTaHeads) {
+    if (tid < nh) {
       my_ml[tid * 2] = -INFINITY;
       my_ml[tid * 2 + 1] = 0.f;
     }
@@ -214,10 +220,10 @@ __global__ void __launch_bounds__(kTaThreads, 1)
   }
   {
     // Q [64 heads x 576] into 8 x 16-byte core matrices: consecutive threads take consecutive heads of one column group
-    const uint16_t *qb = q + (size_t)b * kTaHeads * kTaD;
+    const uint16_t *qb = q + ((size_t)b * heads + h0) * kTaD;
     for (int u = tid; u < kTaHeads * (kTaD / 8); u += kTaThreads) {
       const int kg = u >> 6, h = u & 63;
-      ta_cp16(sQ + kg * kTaLbo + h * 16, qb + (size_t)h * kTaD + kg * 8);
+      ta_cp16(sQ + kg * kTaLbo + h * 16, qb + (size_t)min(h, nh - 1) * kTaD + kg * 8);  // rows past the last head repeat it
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -340,6 +346,16 @@ __global__ void __launch_bounds__(kTaThreads, 1)
             ta_mma(tmem + kTaColO + 64 * j, a_desc + (uint64_t)((2 * j * kTaChunkBytes + kk * 2048) >> 4),
                    p_desc + (uint64_t)(kk * ((2 * kTaLbo) >> 4)), idesc_pv, (n > 0 || kk > 0) ? 1u : 0u);
         }
+        if (FINE) {  // the low parts, in the tile's last chunk
+          const uint64_t lo_desc = ta_desc_plain(sT + buf * kTaTileBytes + (kTaChunks - 1) * kTaChunkBytes, kTaLbo, kTaSbo);
+#pragma unroll
+          for (int kk = 0; kk < kTaTile / 16; ++kk) {
+#pragma unroll
+            for (int j = 0; j < kTaDV / 128; ++j)
+              ta_mma(tmem + kTaColO + 64 * j, a_desc + (uint64_t)((2 * j * kTaChunkBytes + kk * 2048) >> 4),
+                     lo_desc + (uint64_t)(kk * ((2 * kTaLbo) >> 4)), idesc_pv, 1u);
+          }
+        }
         ta_commit(bar_empty + 8 * buf);
         stamp(n, 5);
       };
@@ -381,7 +397,7 @@ __global__ void __launch_bounds__(kTaThreads, 1)
     const int head = 16 * warp + lane;
     for (int n = 0; n < nt; ++n) {
       const int buf = n & 1;
-      uint32_t pk[kTaTile / 2];
+      uint32_t pk[kTaTile / 2], pl[FINE ? kTaTile / 2 : 1];
       bool need = false;
       if (!failed && !ta_wait(bar_sfull + 8 * buf, (uint32_t)((n >> 1) & 1), 6u)) failed = true;
       if (!failed) {
@@ -429,13 +445,23 @@ __global__ void __launch_bounds__(kTaThreads, 1)
 #pragma unroll
         for (int j = 0; j < kTaTile; j += 4) {
           // the probabilities enter the second product rounded to bf16 (as the reference rounds them, :466); the
-          // normaliser sums the same rounded values
-          const uint32_t pa = ta_pack_bf16x2(ta_ex2(fmaf(__uint_as_float(r[j]), sl2, nm)), ta_ex2(fmaf(__uint_as_float(r[j + 1]), sl2, nm)));
-          const uint32_t pb = ta_pack_bf16x2(ta_ex2(fmaf(__uint_as_float(r[j + 2]), sl2, nm)), ta_ex2(fmaf(__uint_as_float(r[j + 3]), sl2, nm)));
-          sum0 += __uint_as_float(pa << 16);
-          sum1 += __uint_as_float(pa & 0xffff0000u);
-          sum2 += __uint_as_float(pb << 16);
-          sum3 += __uint_as_float(pb & 0xffff0000u);
+          // normaliser sums the same rounded values (FINE: two parts, and the normaliser sums the weights themselves)
+          const float p0 = ta_ex2(fmaf(__uint_as_float(r[j]), sl2, nm)), p1 = ta_ex2(fmaf(__uint_as_float(r[j + 1]), sl2, nm));
+          const float p2 = ta_ex2(fmaf(__uint_as_float(r[j + 2]), sl2, nm)), p3 = ta_ex2(fmaf(__uint_as_float(r[j + 3]), sl2, nm));
+          const uint32_t pa = ta_pack_bf16x2(p0, p1), pb = ta_pack_bf16x2(p2, p3);
+          if (FINE) {
+            sum0 += p0;
+            sum1 += p1;
+            sum2 += p2;
+            sum3 += p3;
+            pl[FINE ? j >> 1 : 0] = ta_pack_bf16x2(p0 - __uint_as_float(pa << 16), p1 - __uint_as_float(pa & 0xffff0000u));
+            pl[FINE ? (j >> 1) + 1 : 0] = ta_pack_bf16x2(p2 - __uint_as_float(pb << 16), p3 - __uint_as_float(pb & 0xffff0000u));
+          } else {
+            sum0 += __uint_as_float(pa << 16);
+            sum1 += __uint_as_float(pa & 0xffff0000u);
+            sum2 += __uint_as_float(pb << 16);
+            sum3 += __uint_as_float(pb & 0xffff0000u);
+          }
           pk[j >> 1] = pa;
           pk[(j >> 1) + 1] = pb;
         }
@@ -480,6 +506,13 @@ __global__ void __launch_bounds__(kTaThreads, 1)
 #pragma unroll
             for (int kg = 0; kg < kTaTile / 8; ++kg)
               *reinterpret_cast<uint4 *>(Pp + kg * kTaLbo + head * 16) = make_uint4(pk[4 * kg], pk[4 * kg + 1], pk[4 * kg + 2], pk[4 * kg + 3]);
+            if (FINE) {
+              unsigned char *lo = smem + (size_t)buf * kTaTileBytes + (kTaChunks - 1) * kTaChunkBytes;
+#pragma unroll
+              for (int kg = 0; kg < kTaTile / 8; ++kg)
+                *reinterpret_cast<uint4 *>(lo + kg * kTaLbo + head * 16) =
+                    make_uint4(pl[FINE ? 4 * kg : 0], pl[FINE ? 4 * kg + 1 : 0], pl[FINE ? 4 * kg + 2 : 0], pl[FINE ? 4 * kg + 3 : 0]);
+            }
           }
           asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
           __syncwarp();
@@ -493,7 +526,7 @@ __global__ void __launch_bounds__(kTaThreads, 1)
     failed = ta_consumers_sync(failed);
     if (!failed) {
       tc_fence_after();
-      float *po = part_o + ((size_t)b * splits + split) * kTaHeads * kTaDV;
+      float *po = part_o + (((size_t)b * splits + split) * heads + h0) * kTaDV;
 #pragma unroll 1
       for (int j = 0; j < kTaDV / 128; ++j) {
 #pragma unroll 1
@@ -502,10 +535,11 @@ __global__ void __launch_bounds__(kTaThreads, 1)
           tmem_ld32(tmem + ((uint32_t)(32 * warp) << 16) + kTaColO + 64 * j + 32 * half, o);
           tmem_wait_ld();
 #pragma unroll
-          for (int c = 0; c < 32; ++c) po[(size_t)(32 * half + c) * kTaDV + 128 * j + 32 * warp + lane] = __uint_as_float(o[c]);
+          for (int c = 0; c < 32; ++c)
+            if (32 * half + c < nh) po[(size_t)(32 * half + c) * kTaDV + 128 * j + 32 * warp + lane] = __uint_as_float(o[c]);
         }
       }
-      if (row_ok) {
+      if (row_ok && head < nh) {
         my_ml[head * 2] = m_ref * 0.6931471805599453f;  // back to natural units
         my_ml[head * 2 + 1] = l;
       }
@@ -598,31 +632,44 @@ int launch_mla_attend_tc(const uint16_t *q, const uint16_t *cache, long ctx_stri
                          float scale, float *part_o, float *part_ml, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    BLOK_CUDA(cudaFuncSetAttribute(mla_attend_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTaSmemBytes));
+    BLOK_CUDA(cudaFuncSetAttribute(mla_attend_tc_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTaSmemBytes));
     configured = true;
   }
   CUtensorMap map;
   if (int rc = cache_tensor_map(cache, total_rows, &map)) return rc;
-  mla_attend_tc_kernel<false><<<dim3(splits, B), kTaThreads, kTaSmemBytes, stream>>>(map, q, cache, ctx_stride, seq_len, scale, part_o,
-                                                                                     part_ml, nullptr, nullptr, 0, 0, trace_buffer());
+  mla_attend_tc_kernel<false, false><<<dim3(splits, B), kTaThreads, kTaSmemBytes, stream>>>(map, q, cache, ctx_stride, seq_len, scale, part_o,
+                                                                                     part_ml, nullptr, nullptr, 0, 0, trace_buffer(), kTaHeads);
   return launch_status("mla_attend_tc_kernel");
 }
 
 // The same over a paged pool of pool_rows rows: page_rows must be a positive multiple of the 64-token tile.
-int launch_mla_attend_tc_paged(const uint16_t *q, const uint16_t *pool, long pool_rows, const int *block_table, const int *slot_of,
-                               int table_stride, int page_rows, const int *seq_len, int B, int splits, float scale, float *part_o,
-                               float *part_ml, cudaStream_t stream) {
+template <bool FINE>
+static int launch_paged(const uint16_t *q, const uint16_t *pool, long pool_rows, const int *block_table, const int *slot_of, int table_stride,
+                        int page_rows, const int *seq_len, int B, int heads, int splits, float scale, float *part_o, float *part_ml,
+                        cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    BLOK_CUDA(cudaFuncSetAttribute(mla_attend_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTaSmemBytes));
+    BLOK_CUDA(cudaFuncSetAttribute(mla_attend_tc_kernel<true, FINE>, cudaFuncAttributeMaxDynamicSharedMemorySize, kTaSmemBytes));
     configured = true;
   }
   CUtensorMap map;
   if (int rc = cache_tensor_map(pool, pool_rows, &map)) return rc;
-  mla_attend_tc_kernel<true><<<dim3(splits, B), kTaThreads, kTaSmemBytes, stream>>>(map, q, pool, 0, seq_len, scale, part_o, part_ml,
-                                                                                    block_table, slot_of, table_stride, page_rows,
-                                                                                    trace_buffer());
+  mla_attend_tc_kernel<true, FINE><<<dim3(splits, B, (heads + kTaHeads - 1) / kTaHeads), kTaThreads, kTaSmemBytes, stream>>>(
+      map, q, pool, 0, seq_len, scale, part_o, part_ml, block_table, slot_of, table_stride, page_rows, trace_buffer(), heads);
   return launch_status("mla_attend_tc_kernel(paged)");
+}
+int launch_mla_attend_tc_paged(const uint16_t *q, const uint16_t *pool, long pool_rows, const int *block_table, const int *slot_of,
+                               int table_stride, int page_rows, const int *seq_len, int B, int splits, float scale, float *part_o,
+                               float *part_ml, cudaStream_t stream) {
+  return launch_paged<false>(q, pool, pool_rows, block_table, slot_of, table_stride, page_rows, seq_len, B, kTaHeads, splits, scale, part_o, part_ml,
+                             stream);
+}
+// Any number of heads; the weights in two bf16 parts; entry b attends to rows 0..pos[b].
+int launch_mla_attend_tc_fine(const uint16_t *q, const uint16_t *pool, long pool_rows, const int *block_table, const int *slot_of, int table_stride,
+                              int page_rows, const int *pos, int B, int heads, int splits, float scale, float *part_o, float *part_ml,
+                              cudaStream_t stream) {
+  return launch_paged<true>(q, pool, pool_rows, block_table, slot_of, table_stride, page_rows, pos, B, heads, splits, scale, part_o, part_ml,
+                            stream);
 }
 
 }  // namespace blok

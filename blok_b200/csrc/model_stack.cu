@@ -29,6 +29,8 @@ int launch_bf16_gemv_splitk(const uint16_t *w, const uint16_t *x, uint16_t *y_bf
                             cudaStream_t stream);
 int launch_head_gemv(const uint16_t *w, long w_head_stride, const uint16_t *x, long x_tok_stride, long x_head_stride, uint16_t *y, long y_tok_stride,
                      long y_head_stride, int rows, int cols, int heads, int T, cudaStream_t stream);
+int latent_prompt_take_error(unsigned *out);
+int mla_attend_tc_take_error(unsigned *out);
 int launch_argmax_f32(const float *logits, int vocab, int pitch, int T, uint32_t *ids, cudaStream_t stream);
 
 namespace {
@@ -306,9 +308,14 @@ int load_latent(blok_model *m, Weights &w, const std::string &p, const LatentMix
   s.true_rank = x.kv_rank;
   s.true_q_rank = x.q_rank;
   s.rot_dims = x.rot_dims;
-  s.rot_base = x.rot_base;
   s.scale = (float)x.scale;
   s.eps = (float)S->spec.eps;
+  std::vector<double> turns(x.rot_dims / 2 + 1);
+  for (int i = 0; i < x.rot_dims / 2; ++i) turns[i] = std::pow(x.rot_base, -2.0 * i / x.rot_dims) / 6.28318530717958647693;
+  double *turns_dev = nullptr;
+  TRY(dev_alloc_as(m, turns.size(), &turns_dev));
+  BLOK_CUDA(cudaMemcpy(turns_dev, turns.data(), turns.size() * sizeof(double), cudaMemcpyHostToDevice));
+  s.turns = turns_dev;
   TRY(w.make(&L.dqkv, s.q_rank + s.row(), S->W));
   TRY(w.fill(L.dqkv, 0, p + "dq", Place::plain(x.q_rank, W), fan(W)));
   TRY(w.fill(L.dqkv, s.q_rank, p + "dkv", Place::two_parts(1, x.kv_rank, s.rank, x.rot_dim, s.rot, W), fan(W)));
@@ -368,8 +375,9 @@ int x_map(StackModel *S, const void *x, int cols, const CUtensorMap **out) {
   return BLOK_OK;
 }
 
-// y[T, W.R] = x[T, W.K] W^T; y Act, or fp32 with y_f32.
-int product(StackModel *S, const Mat &w, const void *x, int T, void *y, bool y_f32, cudaStream_t stream) {
+// y[T, W.R] = x[T, W.K] W^T; y Act, or fp32 with y_f32.  silu: *silu columns go through SiLU if the kernel that is picked can
+// do that on the way; *silu becomes 0 then.
+int product(StackModel *S, const Mat &w, const void *x, int T, void *y, bool y_f32, cudaStream_t stream, int *silu = nullptr) {
   if (S->f32) {
     GemmF32 g;
     g.w = w.w;
@@ -395,6 +403,11 @@ int product(StackModel *S, const Mat &w, const void *x, int T, void *y, bool y_f
   g.K = w.K;
   g.out = y;
   g.out_f32 = y_f32;
+  if (silu && *silu) {
+    g.act = GEMM_ACT_SILU;
+    g.act_cols = *silu;
+    *silu = 0;
+  }
   return launch_gemm_tma(g, stream);
 }
 
@@ -576,8 +589,10 @@ struct Call {  // of one step or chunk
 int run_linear(const Call &c, const LinearMixer &x, const LayerState &L, const Run &r) {
   StackModel *S = c.S;
   const int hd = L.lin.heads * L.lin.dim, hv = L.lin.heads * L.lin.vdim;
-  TRY(product(S, L.qkvg, S->h, c.T, S->proj, false, c.stream));
+  int silu = L.lin.silu_qkv ? 2 * hd + hv : 0;
+  TRY(product(S, L.qkvg, S->h, c.T, S->proj, false, c.stream, &silu));
   LinearAttn a = L.lin;
+  a.silu_qkv = silu != 0;
   a.qkvg = S->proj;
   a.ld = L.qkvg.R;
   a.f32 = S->f32;
@@ -807,6 +822,10 @@ int stack_check(blok_model *, blok_stream_t stream) {
   unsigned err = 0;
   TRY(gemm_tma_take_error(&err));
   BLOK_REQUIRE(!err, BLOK_ERR_TIMEOUT, "a product gave up on a barrier");
+  TRY(latent_prompt_take_error(&err));
+  BLOK_REQUIRE(!err, BLOK_ERR_TIMEOUT, "latent attention over a prompt gave up on a barrier");
+  TRY(mla_attend_tc_take_error(&err));
+  BLOK_REQUIRE(!err, BLOK_ERR_TIMEOUT, "the attention core gave up on wait %u", err);
   return BLOK_OK;
 }
 

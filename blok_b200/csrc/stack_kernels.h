@@ -55,7 +55,7 @@ struct LinearAttn {
   const void *qkvg = nullptr;        // Act [T, ld]: q | k | v | g, head by head
   int ld = 0;
   bool f32 = false;
-  bool silu_qkv = false;             // q, k and v go through SiLU (rounded to Act)
+  bool silu_qkv = false;             // q, k and v go through SiLU (rounded to Act) when they are read
   float k_scale = 1.f;
   const float *decay_pow = nullptr;  // [heads, kLinChunk + 1]: decay^i
   float *state = nullptr;            // fp32 [slots, heads, dim, vdim]
@@ -88,7 +88,7 @@ int launch_gated_norm(const GatedNorm &a, int T, cudaStream_t stream);
 struct LatentShape {
   int heads = 0, dim = 0, rot = 0, vdim = 0, rank = 0, q_rank = 0;          // padded
   int true_rot = 0, true_rank = 0, true_q_rank = 0, rot_dims = 0;
-  double rot_base = 1;
+  const double *turns = nullptr;  // device, [rot_dims / 2]: turns per position of every pair, base^(-2i / dims) / 2 pi
   float scale = 1.f, eps = 0.f;
   __host__ __device__ int row() const { return rank + rot; }  // a cached row
   __host__ __device__ int head() const { return dim + rot; }  // a query head

@@ -47,8 +47,8 @@ extern "C" int blok_linear_attention(const void *qkvg, int f32, int ld, int head
 
 extern "C" int blok_gated_norm(const float *o, const void *gate, int ld_gate, const float *w, int heads, int vdim, int true_vdim, int per_head, float eps,
                                int sigmoid, int T, void *out, int ld_out, int f32, blok_stream_t stream) {
-  BLOK_REQUIRE(o && gate && out && T >= 1 && heads >= 1 && vdim % 4 == 0 && true_vdim >= 1 && true_vdim <= vdim && ld_out >= heads * vdim, BLOK_ERR_ARG,
-               "blok_gated_norm: null pointer or bad size");
+  BLOK_REQUIRE(o && gate && out && T >= 1 && heads >= 1 && vdim % 4 == 0 && true_vdim >= 1 && true_vdim <= vdim && ld_gate % 4 == 0 && ld_out % 4 == 0 && ld_out >= heads * vdim,
+               BLOK_ERR_ARG, "blok_gated_norm: null pointer or bad size");
   GatedNorm g;
   g.heads = heads;
   g.vdim = vdim;

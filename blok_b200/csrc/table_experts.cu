@@ -7,7 +7,7 @@
 
 namespace blok {
 
-constexpr int kEpThreads = 256;
+constexpr int kEpThreads = 1024;
 
 __global__ void __launch_bounds__(kEpThreads) expert_plan_kernel(const ExpertPlanArgs *__restrict__ layers, const uint32_t *__restrict__ ids,
                                                                  int vocab, int T) {

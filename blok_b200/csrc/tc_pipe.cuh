@@ -49,6 +49,11 @@ __device__ __forceinline__ void tp_load_2d(uint32_t dst, const CUtensorMap *map,
 __device__ __forceinline__ uint64_t tp_desc_k_sw128(uint32_t saddr) {
   return (uint64_t)((saddr & 0x3FFFFu) >> 4) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
 }
+// MN-major operand in the 128-byte swizzle: 64 contiguous elements of M or N per row, `lead` bytes between 64-element chunks,
+// 1,024 bytes between groups of 8 along K (a K = 16 step advances by 2,048).
+__device__ __forceinline__ uint64_t tp_desc_mn_sw128(uint32_t saddr, uint32_t lead) {
+  return (uint64_t)((saddr & 0x3FFFFu) >> 4) | ((uint64_t)(lead >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
+}
 // bf16 x bf16 -> fp32, M = 128, both operands K-major.
 __host__ __device__ constexpr uint32_t tp_idesc_bf16(int n) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((128u >> 4) << 24);
@@ -60,6 +65,16 @@ __device__ __forceinline__ void tp_mma(uint32_t tmem_d, uint64_t adesc, uint64_t
       "setp.ne.b32 p, %4, 0;\n\t"
       "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
       "}\n" ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+// A from tensor memory (lane = row, two bf16 per 32-bit column, 8 columns per K = 16 step).
+__device__ __forceinline__ void tp_mma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "}\n" ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
 __device__ __forceinline__ void tp_commit(uint32_t mbar) {

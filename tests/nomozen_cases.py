@@ -42,6 +42,8 @@ CASES = {
     # no padding anywhere, sizes of the wide kernels: more than 16 heads, K a multiple of 256, a rank over 256
     "aligned": config(256, 512, 4, [latent(32, 64, 64, 64, 288, 256, mlp=experts(8, 2, 256)),
                                     linear("retention", 4, 128, 128, [0.9, 0.97, 0.99, 0.999], experts(8, 2, 256))]),
+    # the row size of the tcgen05 attention core
+    "core": config(64, 96, 2, [latent(24, 64, 64, 128, 512, 64), latent(70, 32, 64, 16, 512, 32)]),
     # latents too wide for the tensor-core kernel, heads too wide for the prompt kernel
     "wide": config(64, 80, 3, [latent(2, 264, 8, 16, 40, 32), latent(2, 16, 40, 16, 520, 32),
                                linear("lightning", 1, 240, 64, [0.97])]),

@@ -192,12 +192,15 @@ def attend_plain(q, rows, rank, scale, pos):
 
 
 @pytest.mark.parametrize("H,rank,rot,dtype", [(1, 32, 32, torch.bfloat16), (5, 96, 32, torch.bfloat16), (16, 224, 64, torch.bfloat16),
-                                              (40, 512, 64, torch.bfloat16), (17, 160, 32, torch.bfloat16), (3, 544, 32, torch.bfloat16),
+                                              (40, 512, 64, torch.bfloat16), (64, 512, 64, torch.bfloat16), (17, 160, 32, torch.bfloat16), (3, 544, 32, torch.bfloat16),
                                               (6, 96, 32, torch.float32)])
-def test_latent_attend(cuda, H, rank, rot, dtype):
+@pytest.mark.parametrize("core", ["own choice", "mma"])
+def test_latent_attend(cuda, monkeypatch, H, rank, rot, dtype, core):
     """Positions at the edges of tiles, pages and context splits; one key per query stands out somewhere (the first, a far
     one, one at a border, the query's own), so that a lost or foreign row shows at full size."""
     from blok_b200 import lib
+    if core == "mma":
+        monkeypatch.setenv("BLOK_MLA_ATTEND_IMPL", "mma")
     rng = np.random.default_rng(H + rank)
     n, page = 1000, 64
     pos = [0, 1, 62, 63, 64, 65, 127, 128, 129, 500, 640, 998, 999]
@@ -217,7 +220,8 @@ def test_latent_attend(cuda, H, rank, rot, dtype):
         assert np.max(np.abs(got[i] - want[i])) < bar * np.abs(want[i]).max(), p
 
 
-@pytest.mark.parametrize("H,dim,rot,dv", [(1, 32, 32, 16), (3, 64, 32, 64), (2, 64, 64, 128), (2, 128, 64, 112), (2, 192, 64, 256)])
+@pytest.mark.parametrize("H,dim,rot,dv", [(1, 32, 32, 16), (3, 64, 32, 64), (2, 64, 64, 128), (2, 128, 64, 112), (2, 192, 64, 256),
+                                             (2, 128, 64, 128), (3, 64, 64, 64), (1, 192, 64, 128)])
 @pytest.mark.parametrize("T,n", [(33, 33), (200, 200), (64, 321), (129, 128 + 129), (40, 1000)])
 def test_latent_prompt(cuda, H, dim, rot, dv, T, n):
     from blok_b200 import lib
