@@ -108,6 +108,10 @@ constexpr int kLcAhead = 4;  // loads in flight per thread while a tile is stage
 constexpr int kLcCols = 64;  // columns of v per CTA
 constexpr int kLcVPitch = kLcCols * 2 + 16;
 
+__device__ __forceinline__ void lc_wait() {
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+}
 __device__ __forceinline__ uint4 lc_silu8(uint4 v) {
   uint32_t w[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
@@ -115,9 +119,20 @@ __device__ __forceinline__ uint4 lc_silu8(uint4 v) {
   return make_uint4(w[0], w[1], w[2], w[3]);
 }
 
-// `n` rows of `cols` bf16 (a multiple of 8) from p (row pitch ld elements) into a tile; rows past n are zero.
+// `n` rows of `cols` bf16 (a multiple of 8) from p (row pitch ld elements) into a tile; rows past n are zero.  Without SiLU the
+// copies are asynchronous: the caller waits for them.
 __device__ __forceinline__ void lc_stage(unsigned char *dst, int pitch, const uint16_t *p, int ld, int n, int cols, bool silu) {
   const int per = cols / 8, total = kLinChunk * per;
+  if (!silu) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+    for (int u = threadIdx.x; u < total; u += kLcThreads) {
+      const int r = u / per, c = u - r * per;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d + (uint32_t)(r * pitch + c * 16)), "l"(r < n ? p + (size_t)r * ld + c * 8 : p),
+                   "r"(r < n ? 16u : 0u)
+                   : "memory");
+    }
+    return;
+  }
   for (int u0 = threadIdx.x; u0 < total; u0 += kLcAhead * kLcThreads) {
     uint4 v[kLcAhead];
 #pragma unroll
@@ -144,6 +159,7 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_state_kernel(const La
   const float *pw = a.decay_pow + h * (kLinChunk + 1);
   const uint16_t *rows = static_cast<const uint16_t *>(a.qkvg) + (size_t)c * kLinChunk * a.ld;
   const uint16_t *k = rows + (size_t)a.heads * a.dim + (size_t)h * a.dim;
+  lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)a.heads * a.dim + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
   const int per = a.dim / 8, total = kLinChunk * per;
   for (int u0 = threadIdx.x; u0 < total; u0 += kLcAhead * kLcThreads) {  // the decayed keys in three parts
     uint4 x[kLcAhead];
@@ -167,8 +183,7 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_state_kernel(const La
         *reinterpret_cast<uint4 *>(smem + (size_t)(p * kLinChunk + r) * kp + col * 2) = make_uint4(part[0][p], part[1][p], part[2][p], part[3][p]);
     }
   }
-  lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)a.heads * a.dim + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
-  __syncthreads();
+  lc_wait();
   const uint32_t ks = (uint32_t)__cvta_generic_to_shared(smem), vs = (uint32_t)__cvta_generic_to_shared(Vs);
   float *out = a.chunk_state + (((size_t)c * a.heads + h) * a.dim) * a.vdim + v0;
   const int g = lane >> 2, t = lane & 3;
@@ -210,7 +225,7 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LaArgs a) {
   const float *pw = a.decay_pow + h * (kLinChunk + 1);
   float4 *st = reinterpret_cast<float4 *>(a.state + ((size_t)a.slot * a.heads + h) * n + i);
   float4 s = a.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *st;
-  constexpr int kAhead = 4;  // chunks' loads in flight
+  constexpr int kAhead = 8;  // chunks' loads in flight
   const size_t stride = (size_t)a.heads * n / 4;
   float4 *p = reinterpret_cast<float4 *>(a.chunk_state + (size_t)h * n + i);
   for (int c0 = 0; c0 < a.chunks; c0 += kAhead) {
@@ -245,16 +260,17 @@ __global__ void __launch_bounds__(kLcThreads, 2) linear_chunk_out_kernel(const L
   lc_stage(Ks, kp, rows + hd + (size_t)h * a.dim, a.ld, n, a.dim, a.silu);
   lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)hd + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
   const float *S = a.chunk_state + (((size_t)c * a.heads + h) * a.dim) * a.vdim + v0;
+  constexpr int kStateAhead = 8;
   const int per = vc / 4, total = a.dim * per;
-  for (int u0 = threadIdx.x; u0 < total; u0 += kLcAhead * kLcThreads) {  // the state in three parts
-    float4 x[kLcAhead];
+  for (int u0 = threadIdx.x; u0 < total; u0 += kStateAhead * kLcThreads) {  // the state in three parts
+    float4 x[kStateAhead];
 #pragma unroll
-    for (int q = 0; q < kLcAhead; ++q) {
+    for (int q = 0; q < kStateAhead; ++q) {
       const int u = u0 + q * kLcThreads, r = u / per;
       x[q] = u < total ? *reinterpret_cast<const float4 *>(S + (size_t)r * a.vdim + (u - r * per) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
 #pragma unroll
-    for (int q = 0; q < kLcAhead; ++q) {
+    for (int q = 0; q < kStateAhead; ++q) {
       const int u = u0 + q * kLcThreads, r = u / per, col = (u - r * per) * 4;
       if (u >= total) break;
       uint32_t p0[kSplitParts], p1[kSplitParts];
@@ -265,7 +281,7 @@ __global__ void __launch_bounds__(kLcThreads, 2) linear_chunk_out_kernel(const L
         *reinterpret_cast<uint2 *>(Ss + (size_t)(p * a.dim + r) * kLcVPitch + col * 2) = make_uint2(p0[p], p1[p]);
     }
   }
-  __syncthreads();
+  lc_wait();
   const int m0 = (warp & 3) * 16, c0 = (warp >> 2) * (kLcCols / 2);
   if (m0 >= n || c0 >= vc) return;  // no barrier follows
   constexpr int kTiles = kLcCols / 16;  // the warp's column tiles of 8
