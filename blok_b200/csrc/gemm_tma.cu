@@ -42,7 +42,7 @@ __device__ __forceinline__ float gt_act(float v) {
     v = fmaxf(v, 0.f);
     return v * v;
   }
-  if (ACT == GEMM_ACT_SILU) return v / (1.0f + expf(-v));
+  if (ACT == GEMM_ACT_SILU) return __fdividef(v, 1.0f + __expf(-v));  // the result is rounded to bf16
   return v;
 }
 
