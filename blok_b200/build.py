@@ -21,8 +21,9 @@ OBJ = os.path.join(HERE, "build")
 CLI = os.path.join(HERE, "blok-kimi-exec")
 TRACE_RUN = os.path.join(HERE, "blok-trace-run")
 # What a model opened from a config.json needs: blok-trace-run is linked from these objects alone.
-STACK_SOURCES = ["abi", "batcher", "bf16_kernels", "gemm_f32", "gemm_tma", "kv_pages", "latent_attn", "latent_prompt_tc", "linear_attn", "lm_head",
-                 "mla_attend_tc", "model", "model_stack", "nomozen", "residual_streams", "table_experts", "wgemm_stream"]
+STACK_SOURCES = ["abi", "batcher", "bf16_kernels", "gemm_f32", "gemm_tma", "grouped_attn", "kv_pages", "latent_attn", "linear_attn", "lm_head",
+                 "mla_attend_tc", "model", "model_stack", "nomozen", "pamopel", "prompt_attn_tc", "residual_norm", "residual_streams", "state_space",
+                 "table_experts", "wgemm_stream"]
 
 NVCC_FLAGS = [
     "-std=c++17", "-O3", "-lineinfo", "-gencode", "arch=compute_100a,code=sm_100a",

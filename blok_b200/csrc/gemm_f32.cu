@@ -48,4 +48,19 @@ int launch_gemm_f32(const GemmF32 &g, cudaStream_t stream) {
   return launch_status("gemm_f32_kernel");
 }
 
+// out[t, r] = silu(x[t, r]) * x[t, cols + r]
+__global__ void __launch_bounds__(256) swiglu_f32_kernel(const float *__restrict__ x, float *__restrict__ out, int cols, long n) {
+  const long i = (long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= n) return;
+  const float *p = x + i / cols * 2 * cols + i % cols;
+  const float z = p[0];
+  out[i] = z / (1.0f + expf(-z)) * p[cols];
+}
+
+int launch_swiglu_f32(const float *x, float *out, int cols, int T, cudaStream_t stream) {
+  const long n = (long)cols * T;
+  swiglu_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>(x, out, cols, n);
+  return launch_status("swiglu_f32_kernel");
+}
+
 }  // namespace blok

@@ -33,7 +33,7 @@ __device__ unsigned g_gemm_tma_error = 0;
 struct GtArgs {
   void *out;
   const int *tile_expert, *tile_start, *tile_count, *num_tiles;
-  int T, R, K, ldo, act_cols;
+  int T, R, K, ldo, act_cols, up_row;
 };
 
 template <int ACT>
@@ -51,11 +51,13 @@ __global__ void __launch_bounds__(kGtThreads)
     gemm_tma_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ CUtensorMap mw, const GtArgs a) {
   using Cfg = GtCfg<BN>;
   constexpr int S = Cfg::kStages;
+  // a pair of 128-row boxes, gate and up, makes 128 output columns
+  constexpr int kCols = ACT == GEMM_ACT_SWIGLU ? BN / 2 : BN;
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(8) unsigned long long s_bar[2 * S + 1];
   __shared__ uint32_t s_tmem;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  int row0, count, wrow = blockIdx.x * BN;
+  int row0, count, wrow = blockIdx.x * kCols;
   if (a.tile_start) {
     if ((int)blockIdx.y >= *a.num_tiles) return;
     row0 = a.tile_start[blockIdx.y];
@@ -98,6 +100,7 @@ __global__ void __launch_bounds__(kGtThreads)
         tp_expect_tx(full + 8 * s, Cfg::kStageBytes);
         tp_load_2d(dst, &mx, c * kGtKStep, row0, full + 8 * s);
         tp_load_2d(dst + Cfg::kABytes, &mw, c * kGtKStep, wrow, full + 8 * s);
+        if (ACT == GEMM_ACT_SWIGLU) tp_load_2d(dst + Cfg::kABytes + kCols * 128, &mw, c * kGtKStep, a.up_row + wrow, full + 8 * s);
         issued = c + 1;
       }
       // no copy may be in flight when the CTA leaves; the MMA lane has seen all of them unless a wait gave up
@@ -128,7 +131,30 @@ __global__ void __launch_bounds__(kGtThreads)
       tc_fence_after();
       const int r = 32 * warp + lane;
       const size_t o = (size_t)(row0 + r) * a.ldo;
-      const int n0 = blockIdx.x * BN;
+      const int n0 = blockIdx.x * kCols;
+      if constexpr (ACT == GEMM_ACT_SWIGLU) {
+#pragma unroll 1
+        for (int c0 = 0; c0 < kCols; c0 += 16) {
+          if (n0 + c0 >= a.R) break;
+          uint32_t gate[16], up[16];
+          const uint32_t at = tmem + ((uint32_t)(32 * warp) << 16) + c0;
+          tmem_ld16(at, gate);
+          tmem_ld16(at + kCols, up);
+          tmem_wait_ld();
+          if (r < count) {
+#pragma unroll
+            for (int j = 0; j < 16; j += 4) {
+              const int col = n0 + c0 + j;
+              if (col < a.R) {
+                float f[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) f[i] = gt_act<GEMM_ACT_SILU>(__uint_as_float(gate[j + i])) * __uint_as_float(up[j + i]);
+                *reinterpret_cast<uint2 *>(static_cast<uint16_t *>(a.out) + o + col) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+              }
+            }
+          }
+        }
+      } else
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += 32) {
         if (n0 + c0 >= a.R) break;
@@ -185,14 +211,18 @@ int gemm_operand_map(const void *base, long rows, int cols, long pitch, int box,
 
 template <int BN, int ACT, bool F32>
 static int gt_launch(const GemmTma &g, dim3 grid, cudaStream_t stream) {
-  const GtArgs a = {g.out, g.tile_expert, g.tile_start, g.tile_count, g.num_tiles, g.T, g.R, g.K, g.ldo, g.act_cols};
+  const GtArgs a = {g.out, g.tile_expert, g.tile_start, g.tile_count, g.num_tiles, g.T, g.R, g.K, g.ldo, g.act_cols, g.up_row};
   BLOK_CUDA(cudaFuncSetAttribute(gemm_tma_kernel<BN, ACT, F32>, cudaFuncAttributeMaxDynamicSharedMemorySize, GtCfg<BN>::kSmem));
-  gemm_tma_kernel<BN, ACT, F32><<<grid, kGtThreads, GtCfg<BN>::kSmem, stream>>>(*g.x, BN == 128 ? *g.w128 : *g.w256, a);
+  gemm_tma_kernel<BN, ACT, F32><<<grid, kGtThreads, GtCfg<BN>::kSmem, stream>>>(*g.x, BN == 128 || ACT == GEMM_ACT_SWIGLU ? *g.w128 : *g.w256, a);
   return launch_status("gemm_tma_kernel");
 }
 
 int launch_gemm_tma(const GemmTma &g, cudaStream_t stream) {
   BLOK_REQUIRE(g.x && g.w128 && g.out && g.R % 4 == 0 && g.K % 8 == 0 && g.T >= 1, BLOK_ERR_SHAPE, "gemm: T %d, R %d, K %d", g.T, g.R, g.K);
+  if (g.act == GEMM_ACT_SWIGLU) {
+    BLOK_REQUIRE(!g.out_f32 && !g.tile_start, BLOK_ERR_SHAPE, "gemm: a gated product is bf16 and not grouped");
+    return gt_launch<256, GEMM_ACT_SWIGLU, false>(g, dim3((g.R + 127) / 128, (g.T + kGtTileRows - 1) / kGtTileRows), stream);
+  }
   const int tiles = g.tile_start ? g.max_tiles : (g.T + kGtTileRows - 1) / kGtTileRows;
   // the wide tile reads fewer bytes from shared memory per product; it needs enough tiles to fill the GPU
   const long wide = (long)((g.R + 255) / 256) * (g.tile_start ? (g.T + kGtTileRows - 1) / kGtTileRows : tiles);

@@ -7,7 +7,7 @@
 
 namespace blok {
 
-enum { GEMM_ACT_NONE = 0, GEMM_ACT_RELU2 = 1, GEMM_ACT_SILU = 2 };
+enum { GEMM_ACT_NONE = 0, GEMM_ACT_RELU2 = 1, GEMM_ACT_SILU = 2, GEMM_ACT_SWIGLU = 3 };
 constexpr int kGtTileRows = 128;  // rows of x per tile
 
 // A matrix operand: bf16 [rows, cols], rows `pitch` elements apart (pitch a multiple of 8, base 16-byte aligned).
@@ -24,6 +24,8 @@ struct GemmTma {
   int ldo = 0;
   int act = GEMM_ACT_NONE;
   int act_cols = 0;                            // GEMM_ACT_SILU: the first so many columns (a multiple of 4) only; bf16 output
+  // GEMM_ACT_SWIGLU: out[t, r] = silu(row r) * (row up_row + r), bf16 (R counts the outputs; the weights hold both halves)
+  int up_row = 0;
   // Grouped form: tile i covers rows [tile_start[i], + tile_count[i]) of x (at most kGtTileRows) and weight rows
   // [tile_expert[i] * R, + R); at most max_tiles tiles, *num_tiles of them valid.  NULL: consecutive tiles of one matrix.
   const int *tile_expert = nullptr, *tile_start = nullptr, *tile_count = nullptr, *num_tiles = nullptr;

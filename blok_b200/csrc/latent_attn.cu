@@ -4,7 +4,7 @@
 // Two forms, both causal.  Absorbed (decode, short portions): queries multiplied by W_UK^T score against the cached rows
 // themselves and the latents are averaged, one pass over the cache, the context split over CTAs (mla_merge.cuh adds the
 // parts).  Prompt form (long portions): per-head keys and values are made from the cached latents by one product and a
-// tile kernel walks them, which needs 3 to 4 times fewer multiply-adds per query and key (latent_prompt_tc.cu on tcgen05 for
+// tile kernel walks them, which needs 3 to 4 times fewer multiply-adds per query and key (prompt_attn_tc.cu on tcgen05 for
 // sizes in multiples of 64, the mma.sync kernel here for the others).
 //
 // Scores, softmax and its weights are fp32; the weights enter the second product in three bf16 parts (bf16_split.cuh).

@@ -1,12 +1,15 @@
-// Linear attention with a fixed decay per head and no softmax (retention, lightning attention):
-//   S_t = decay S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t                     (S fp32 [dim, vdim], per head and sequence)
+// Linear attention without a softmax:
+//   S_t = decay_t S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t                   (S fp32 [dim, vdim], per head and sequence)
+// with a fixed decay per head (retention, lightning attention), or with a decay and a key scale per head and token and a
+// skip o_t += D v_t (a selective state space: q = C, k = dt B, v = x, shared by several heads; state_space.cu makes them).
 //
 // Decode runs the recurrence itself, every thread holding a few elements of S in registers.  A prompt runs in chunks of 64
 // tokens: with w_ij = decay^(i-j) for j <= i inside a chunk and S the state in front of it,
 //   o_i = sum_j w_ij (q_i . k_j) v_j + decay^(i+1) S^T q_i
 //   S'  = decay^L S + sum_j decay^(L-1-j) k_j v_j^T                        (L tokens in the chunk)
 // in three launches: every chunk's own contribution to the state in parallel, a scan over the chunks that turns the
-// contributions into the states in front of them, every chunk's output in parallel.  The products run on bf16 tensor cores
+// contributions into the states in front of them, every chunk's output in parallel.  With decays per token every power becomes
+// the exponential of a difference of the logarithms' running sums, which are kept in two fp32 parts.  The products run on bf16 tensor cores
 // with their fp32 factors (scores, decays, states) split into three bf16 parts (bf16_split.cuh).
 #include "bf16_split.cuh"
 #include "stack_kernels.h"
@@ -28,8 +31,12 @@ __device__ __forceinline__ float la_proj(const Act *p, bool silu) {
 }
 
 struct LaArgs {
-  const void *qkvg;
+  const void *q, *k, *v;  // a token's rows: heads / share heads of q and k, heads of v; `ld` values between tokens
+  int share;
   const float *decay_pow;
+  const float4 *token;    // decays per token: [heads, token_ld] of (key scale, log decay, running sum of the log decays in two parts)
+  int token_ld;
+  const float *skip;      // with token: [heads]
   float *state, *o, *chunk_state;
   const int *slot_of, *pos;  // step form
   int slot;                  // chunk form
@@ -40,7 +47,7 @@ struct LaArgs {
 
 // ---- the recurrence: T tokens of each of gridDim.z sequences, one after the other.  CTA = 32 columns of a head's state,
 // thread = 4 columns x every 32nd row. ----
-template <typename Act, int R>
+template <typename Act, int R, bool TOKEN>
 __global__ void __launch_bounds__(256) linear_recurrent_kernel(const LaArgs a) {
   __shared__ float sq[32 * R], sk[32 * R];
   __shared__ float4 s_red[8][8];
@@ -49,8 +56,8 @@ __global__ void __launch_bounds__(256) linear_recurrent_kernel(const LaArgs a) {
   const bool in_col = col < a.vdim;
   const int slot = a.slot_of ? a.slot_of[b] : a.slot;
   const bool fresh = a.slot_of ? a.pos[b] == 0 : a.fresh != 0;
-  const float decay = a.decay_pow[h * (kLinChunk + 1) + 1];
-  const int hd = a.heads * a.dim;
+  float decay = TOKEN ? 0.f : a.decay_pow[h * (kLinChunk + 1) + 1], k_scale = a.k_scale;
+  const float skip = TOKEN ? a.skip[h] : 0.f;
   float *st = a.state + ((size_t)slot * a.heads + h) * a.dim * a.vdim + col;
   float4 s[R];
 #pragma unroll
@@ -60,15 +67,20 @@ __global__ void __launch_bounds__(256) linear_recurrent_kernel(const LaArgs a) {
   }
   for (int t = 0; t < a.T; ++t) {
     const size_t row = (size_t)b * a.T + t;
-    const Act *p = static_cast<const Act *>(a.qkvg) + row * a.ld + (size_t)h * a.dim;
+    const size_t qk = row * a.ld + (size_t)(h / a.share) * a.dim + tid;
+    if (TOKEN) {
+      const float4 w = a.token[(size_t)h * a.token_ld + row];
+      k_scale = w.x;
+      decay = expf(w.y);
+    }
     if (tid < 32 * R) {
       const bool in = tid < a.dim;
-      sq[tid] = in ? la_proj(p + tid, a.silu) : 0.f;
-      sk[tid] = in ? la_proj(p + hd + tid, a.silu) * a.k_scale : 0.f;
+      sq[tid] = in ? la_proj(static_cast<const Act *>(a.q) + qk, a.silu) : 0.f;
+      sk[tid] = in ? la_proj(static_cast<const Act *>(a.k) + qk, a.silu) * k_scale : 0.f;
     }
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (in_col) {
-      const Act *pv = static_cast<const Act *>(a.qkvg) + row * a.ld + 2 * (size_t)hd + (size_t)h * a.vdim + col;
+      const Act *pv = static_cast<const Act *>(a.v) + row * a.ld + (size_t)h * a.vdim + col;
       v = make_float4(la_proj(pv, a.silu), la_proj(pv + 1, a.silu), la_proj(pv + 2, a.silu), la_proj(pv + 3, a.silu));
     }
     __syncthreads();
@@ -92,6 +104,7 @@ __global__ void __launch_bounds__(256) linear_recurrent_kernel(const LaArgs a) {
       float4 u = s_red[0][tid];
 #pragma unroll
       for (int w = 1; w < 8; ++w) u = make_float4(u.x + s_red[w][tid].x, u.y + s_red[w][tid].y, u.z + s_red[w][tid].z, u.w + s_red[w][tid].w);
+      if (TOKEN) u = make_float4(fmaf(skip, v.x, u.x), fmaf(skip, v.y, u.y), fmaf(skip, v.z, u.z), fmaf(skip, v.w, u.w));
       *reinterpret_cast<float4 *>(a.o + row * a.heads * a.vdim + (size_t)h * a.vdim + col) = u;
     }
   }
@@ -148,18 +161,36 @@ __device__ __forceinline__ void lc_stage(unsigned char *dst, int pitch, const ui
   }
 }
 
+// exp(a - b) of running sums in two parts
+__device__ __forceinline__ float lc_between(float4 a, float4 b) { return expf((a.z - b.z) + (a.w - b.w)); }
+
 // chunk_state[c][h] = sum_j k_scale decay^(L-1-j) k_j v_j^T.  grid = (chunks, heads, columns / 64)
+template <bool TOKEN>
 __global__ void __launch_bounds__(kLcThreads) linear_chunk_state_kernel(const LaArgs a) {
   extern __shared__ __align__(16) unsigned char smem[];
+  __shared__ float s_wt[kLinChunk];
   const int c = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * kLcCols;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int n = min(kLinChunk, a.T - c * kLinChunk), vc = min(kLcCols, a.vdim - v0);
   const int kp = a.dim * 2 + 16;  // pitch of the key tiles
   unsigned char *Vs = smem + (size_t)kSplitParts * kLinChunk * kp;
-  const float *pw = a.decay_pow + h * (kLinChunk + 1);
-  const uint16_t *rows = static_cast<const uint16_t *>(a.qkvg) + (size_t)c * kLinChunk * a.ld;
-  const uint16_t *k = rows + (size_t)a.heads * a.dim + (size_t)h * a.dim;
-  lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)a.heads * a.dim + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
+  const size_t rows = (size_t)c * kLinChunk * a.ld;
+  const uint16_t *k = static_cast<const uint16_t *>(a.k) + rows + (size_t)(h / a.share) * a.dim;
+  lc_stage(Vs, kLcVPitch, static_cast<const uint16_t *>(a.v) + rows + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
+  if (threadIdx.x < kLinChunk) {
+    const int r = threadIdx.x;
+    float wt = 0.f;
+    if (r < n) {
+      if (TOKEN) {
+        const float4 *tok = a.token + (size_t)h * a.token_ld + c * kLinChunk;
+        wt = tok[r].x * lc_between(tok[n - 1], tok[r]);
+      } else {
+        wt = a.k_scale * a.decay_pow[h * (kLinChunk + 1) + n - 1 - r];
+      }
+    }
+    s_wt[r] = wt;
+  }
+  __syncthreads();
   const int per = a.dim / 8, total = kLinChunk * per;
   for (int u0 = threadIdx.x; u0 < total; u0 += kLcAhead * kLcThreads) {  // the decayed keys in three parts
     uint4 x[kLcAhead];
@@ -173,7 +204,7 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_state_kernel(const La
       const int u = u0 + q * kLcThreads, r = u / per, col = (u - r * per) * 8;
       if (u >= total) break;
       if (a.silu) x[q] = lc_silu8(x[q]);
-      const float wt = r < n ? a.k_scale * pw[n - 1 - r] : 0.f;
+      const float wt = s_wt[r];
       const uint32_t w[4] = {x[q].x, x[q].y, x[q].z, x[q].w};
       uint32_t part[4][kSplitParts];
 #pragma unroll
@@ -219,10 +250,10 @@ __global__ void __launch_bounds__(kLcThreads) linear_chunk_state_kernel(const La
 }
 
 // chunk_state[c] <- the state in front of chunk c; state <- the state behind the last chunk.
+template <bool TOKEN>
 __global__ void __launch_bounds__(128) linear_scan_kernel(const LaArgs a) {
   const int h = blockIdx.y, i = (blockIdx.x * blockDim.x + threadIdx.x) * 4, n = a.dim * a.vdim;
   if (i >= n) return;
-  const float *pw = a.decay_pow + h * (kLinChunk + 1);
   float4 *st = reinterpret_cast<float4 *>(a.state + ((size_t)a.slot * a.heads + h) * n + i);
   float4 s = a.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *st;
   constexpr int kAhead = 8;  // chunks' loads in flight
@@ -236,7 +267,14 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LaArgs a) {
 #pragma unroll
     for (int j = 0; j < kAhead; ++j)
       if (c0 + j < a.chunks) {
-        const float d = pw[min(kLinChunk, a.T - (c0 + j) * kLinChunk)];
+        const int n = min(kLinChunk, a.T - (c0 + j) * kLinChunk);
+        float d;
+        if (TOKEN) {
+          const float4 w = a.token[(size_t)h * a.token_ld + (c0 + j) * kLinChunk + n - 1];
+          d = expf(w.z + w.w);
+        } else {
+          d = a.decay_pow[h * (kLinChunk + 1) + n];
+        }
         p[(size_t)(c0 + j) * stride] = s;
         s = make_float4(fmaf(d, s.x, own[j].x), fmaf(d, s.y, own[j].y), fmaf(d, s.z, own[j].z), fmaf(d, s.w, own[j].w));
       }
@@ -245,20 +283,26 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LaArgs a) {
 }
 
 // grid = (chunks, heads, columns / 64); a warp owns 16 tokens of the chunk and half of the columns.
+template <bool TOKEN>
 __global__ void __launch_bounds__(kLcThreads, 2) linear_chunk_out_kernel(const LaArgs a) {
   extern __shared__ __align__(16) unsigned char smem[];
-  __shared__ float s_pw[kLinChunk + 1];
+  __shared__ float s_pw[TOKEN ? 1 : kLinChunk + 1];
+  __shared__ float4 s_tok[TOKEN ? kLinChunk : 1];
   const int c = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * kLcCols;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
   const int n = min(kLinChunk, a.T - c * kLinChunk), vc = min(kLcCols, a.vdim - v0);
   const int kp = a.dim * 2 + 16;
   unsigned char *Ks = smem + (size_t)kLinChunk * kp, *Vs = Ks + (size_t)kLinChunk * kp, *Ss = Vs + (size_t)kLinChunk * kLcVPitch;
-  const uint16_t *rows = static_cast<const uint16_t *>(a.qkvg) + (size_t)c * kLinChunk * a.ld;
-  const int hd = a.heads * a.dim;
-  if (threadIdx.x <= kLinChunk) s_pw[threadIdx.x] = a.decay_pow[h * (kLinChunk + 1) + threadIdx.x];
-  lc_stage(smem, kp, rows + (size_t)h * a.dim, a.ld, n, a.dim, a.silu);
-  lc_stage(Ks, kp, rows + hd + (size_t)h * a.dim, a.ld, n, a.dim, a.silu);
-  lc_stage(Vs, kLcVPitch, rows + 2 * (size_t)hd + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
+  const size_t qk = (size_t)c * kLinChunk * a.ld + (size_t)(h / a.share) * a.dim;
+  if (TOKEN) {
+    if (threadIdx.x < kLinChunk)
+      s_tok[threadIdx.x] = threadIdx.x < n ? a.token[(size_t)h * a.token_ld + c * kLinChunk + threadIdx.x] : make_float4(0.f, 0.f, 0.f, 0.f);
+  } else if (threadIdx.x <= kLinChunk) {
+    s_pw[threadIdx.x] = a.decay_pow[h * (kLinChunk + 1) + threadIdx.x];
+  }
+  lc_stage(smem, kp, static_cast<const uint16_t *>(a.q) + qk, a.ld, n, a.dim, a.silu);
+  lc_stage(Ks, kp, static_cast<const uint16_t *>(a.k) + qk, a.ld, n, a.dim, a.silu);
+  lc_stage(Vs, kLcVPitch, static_cast<const uint16_t *>(a.v) + (size_t)c * kLinChunk * a.ld + (size_t)h * a.vdim + v0, a.ld, n, vc, a.silu);
   const float *S = a.chunk_state + (((size_t)c * a.heads + h) * a.dim) * a.vdim + v0;
   constexpr int kStateAhead = 8;
   const int per = vc / 4, total = a.dim * per;
@@ -314,7 +358,14 @@ __global__ void __launch_bounds__(kLcThreads, 2) linear_chunk_out_kernel(const L
     }
   }
   // the state's share decays by one step more than the token's place in the chunk
-  const float d_lo = s_pw[m0 + g + 1], d_hi = s_pw[m0 + g + 9];
+  float d_lo, d_hi;
+  float4 k_lo, k_hi;  // the tokens' own entries
+  if (TOKEN) {
+    k_lo = s_tok[m0 + g], k_hi = s_tok[m0 + g + 8];
+    d_lo = expf(k_lo.z + k_lo.w), d_hi = expf(k_hi.z + k_hi.w);
+  } else {
+    d_lo = s_pw[m0 + g + 1], d_hi = s_pw[m0 + g + 9];
+  }
 #pragma unroll
   for (int nt = 0; nt < kTiles; ++nt) {
     acc[nt][0] *= d_lo;
@@ -331,8 +382,15 @@ __global__ void __launch_bounds__(kLcThreads, 2) linear_chunk_out_kernel(const L
       for (int half = 0; half < 2; ++half) {
         const float *s = sc[2 * kk + half];
         const int j = kk * 16 + half * 8 + 2 * t;
-        const float w0 = j <= i_lo ? s[0] * a.k_scale * s_pw[i_lo - j] : 0.f, w1 = j + 1 <= i_lo ? s[1] * a.k_scale * s_pw[i_lo - j - 1] : 0.f;
-        const float w2 = j <= i_hi ? s[2] * a.k_scale * s_pw[i_hi - j] : 0.f, w3 = j + 1 <= i_hi ? s[3] * a.k_scale * s_pw[i_hi - j - 1] : 0.f;
+        float w0, w1, w2, w3;
+        if (TOKEN) {
+          const float4 a0 = s_tok[j], a1 = s_tok[j + 1];
+          w0 = j <= i_lo ? s[0] * a0.x * lc_between(k_lo, a0) : 0.f, w1 = j + 1 <= i_lo ? s[1] * a1.x * lc_between(k_lo, a1) : 0.f;
+          w2 = j <= i_hi ? s[2] * a0.x * lc_between(k_hi, a0) : 0.f, w3 = j + 1 <= i_hi ? s[3] * a1.x * lc_between(k_hi, a1) : 0.f;
+        } else {
+          w0 = j <= i_lo ? s[0] * a.k_scale * s_pw[i_lo - j] : 0.f, w1 = j + 1 <= i_lo ? s[1] * a.k_scale * s_pw[i_lo - j - 1] : 0.f;
+          w2 = j <= i_hi ? s[2] * a.k_scale * s_pw[i_hi - j] : 0.f, w3 = j + 1 <= i_hi ? s[3] * a.k_scale * s_pw[i_hi - j - 1] : 0.f;
+        }
         split_pair(w0, w1, fa[2 * half]);
         split_pair(w2, w3, fa[2 * half + 1]);
       }
@@ -347,6 +405,20 @@ __global__ void __launch_bounds__(kLcThreads, 2) linear_chunk_out_kernel(const L
             mma_bf16_16816(acc[nt + 1], fa[0][p], fa[1][p], fa[2][p], fa[3][p], b2, b3);
           }
         }
+      }
+    }
+  }
+  if (TOKEN) {
+    const float skip = a.skip[h];
+#pragma unroll
+    for (int nt = 0; nt < kTiles; ++nt) {
+      if (c0 + nt * 8 < vc) {
+        const unsigned char *v = Vs + (size_t)i_lo * kLcVPitch + (c0 + nt * 8 + 2 * t) * 2;
+        const uint32_t lo = *reinterpret_cast<const uint32_t *>(v), hi = *reinterpret_cast<const uint32_t *>(v + 8 * kLcVPitch);
+        acc[nt][0] = fmaf(skip, bf16lo(lo), acc[nt][0]);
+        acc[nt][1] = fmaf(skip, bf16hi(lo), acc[nt][1]);
+        acc[nt][2] = fmaf(skip, bf16lo(hi), acc[nt][2]);
+        acc[nt][3] = fmaf(skip, bf16hi(hi), acc[nt][3]);
       }
     }
   }
@@ -468,7 +540,15 @@ int launch_gated_norm(const GatedNorm &a, int T, cudaStream_t stream) {
 
 static LaArgs la_args(const LinearAttn &a) {
   LaArgs r{};
-  r.qkvg = a.qkvg;
+  const size_t esz = a.f32 ? 4 : 2, hd = (size_t)a.heads / a.share * a.dim;
+  const char *p = static_cast<const char *>(a.qkvg);
+  r.q = p + (a.v_first ? ((size_t)a.heads * a.vdim + hd) * esz : 0);
+  r.k = p + (a.v_first ? (size_t)a.heads * a.vdim : hd) * esz;
+  r.v = p + (a.v_first ? 0 : 2 * hd * esz);
+  r.share = a.share;
+  r.token = a.token;
+  r.token_ld = a.token_ld;
+  r.skip = a.skip;
   r.decay_pow = a.decay_pow;
   r.state = a.state;
   r.o = a.o;
@@ -482,16 +562,21 @@ static LaArgs la_args(const LinearAttn &a) {
   return r;
 }
 
+template <typename Act, bool TOKEN>
+static int recurrent_of(const LaArgs &r, int seqs, cudaStream_t stream) {
+  const dim3 grid((r.vdim + 31) / 32, r.heads, seqs);
+  if (r.dim <= 64) linear_recurrent_kernel<Act, 2, TOKEN><<<grid, 256, 0, stream>>>(r);
+  else if (r.dim <= 128) linear_recurrent_kernel<Act, 4, TOKEN><<<grid, 256, 0, stream>>>(r);
+  else linear_recurrent_kernel<Act, 8, TOKEN><<<grid, 256, 0, stream>>>(r);
+  return launch_status("linear_recurrent_kernel");
+}
 template <typename Act>
 static int recurrent(const LaArgs &r, int seqs, cudaStream_t stream) {
-  const dim3 grid((r.vdim + 31) / 32, r.heads, seqs);
-  if (r.dim <= 64) linear_recurrent_kernel<Act, 2><<<grid, 256, 0, stream>>>(r);
-  else if (r.dim <= 128) linear_recurrent_kernel<Act, 4><<<grid, 256, 0, stream>>>(r);
-  else linear_recurrent_kernel<Act, 8><<<grid, 256, 0, stream>>>(r);
-  return launch_status("linear_recurrent_kernel");
+  return r.token ? recurrent_of<Act, true>(r, seqs, stream) : recurrent_of<Act, false>(r, seqs, stream);
 }
 
 static int check_shape(const LinearAttn &a) {
+  BLOK_REQUIRE(a.share >= 1 && a.heads % a.share == 0 && (!a.token || a.skip), BLOK_ERR_SHAPE, "linear attention: %d heads, %d to a key", a.heads, a.share);
   BLOK_REQUIRE(a.heads >= 1 && a.dim >= 16 && a.dim % 16 == 0 && a.dim <= kLinMaxDim && a.vdim >= 16 && a.vdim % 16 == 0 && a.ld % 8 == 0,
                BLOK_ERR_SHAPE, "linear attention: %d heads of %d x %d (a head's key size is at most %d)", a.heads, a.dim, a.vdim, kLinMaxDim);
   return BLOK_OK;
@@ -510,6 +595,22 @@ size_t linear_chunk_scratch_bytes(int heads, int dim, int vdim, int T) {
   return (size_t)((T + kLinChunk - 1) / kLinChunk) * heads * dim * vdim * sizeof(float);
 }
 
+template <bool TOKEN>
+static int chunked(const LaArgs &r, cudaStream_t stream) {
+  const int kp = r.dim * 2 + 16;
+  const dim3 grid(r.chunks, r.heads, (r.vdim + kLcCols - 1) / kLcCols);
+  const size_t smem1 = (size_t)kSplitParts * kLinChunk * kp + (size_t)kLinChunk * kLcVPitch;
+  const size_t smem3 = (size_t)2 * kLinChunk * kp + (size_t)kLinChunk * kLcVPitch + (size_t)kSplitParts * r.dim * kLcVPitch;
+  BLOK_CUDA(cudaFuncSetAttribute(linear_chunk_state_kernel<TOKEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1));
+  BLOK_CUDA(cudaFuncSetAttribute(linear_chunk_out_kernel<TOKEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3));
+  linear_chunk_state_kernel<TOKEN><<<grid, kLcThreads, smem1, stream>>>(r);
+  if (int rc = launch_status("linear_chunk_state_kernel")) return rc;
+  linear_scan_kernel<TOKEN><<<dim3((r.dim * r.vdim / 4 + 127) / 128, r.heads), 128, 0, stream>>>(r);
+  if (int rc = launch_status("linear_scan_kernel")) return rc;
+  linear_chunk_out_kernel<TOKEN><<<grid, kLcThreads, smem3, stream>>>(r);
+  return launch_status("linear_chunk_out_kernel");
+}
+
 int launch_linear_chunk(const LinearAttn &a, int slot, long first_pos, int T, cudaStream_t stream) {
   if (int rc = check_shape(a)) return rc;
   LaArgs r = la_args(a);
@@ -519,18 +620,7 @@ int launch_linear_chunk(const LinearAttn &a, int slot, long first_pos, int T, cu
   if (a.f32) return recurrent<float>(r, 1, stream);
   if (T <= 8) return recurrent<uint16_t>(r, 1, stream);
   r.chunks = (T + kLinChunk - 1) / kLinChunk;
-  const int kp = a.dim * 2 + 16;
-  const dim3 grid(r.chunks, a.heads, (a.vdim + kLcCols - 1) / kLcCols);
-  const size_t smem1 = (size_t)kSplitParts * kLinChunk * kp + (size_t)kLinChunk * kLcVPitch;
-  const size_t smem3 = (size_t)2 * kLinChunk * kp + (size_t)kLinChunk * kLcVPitch + (size_t)kSplitParts * a.dim * kLcVPitch;
-  BLOK_CUDA(cudaFuncSetAttribute(linear_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1));
-  BLOK_CUDA(cudaFuncSetAttribute(linear_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3));
-  linear_chunk_state_kernel<<<grid, kLcThreads, smem1, stream>>>(r);
-  if (int rc = launch_status("linear_chunk_state_kernel")) return rc;
-  linear_scan_kernel<<<dim3((a.dim * a.vdim / 4 + 127) / 128, a.heads), 128, 0, stream>>>(r);
-  if (int rc = launch_status("linear_scan_kernel")) return rc;
-  linear_chunk_out_kernel<<<grid, kLcThreads, smem3, stream>>>(r);
-  return launch_status("linear_chunk_out_kernel");
+  return a.token ? chunked<true>(r, stream) : chunked<false>(r, stream);
 }
 
 }  // namespace blok

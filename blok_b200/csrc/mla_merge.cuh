@@ -1,4 +1,4 @@
-// The merge behind the split-context attention cores (mla.cu, latent_attn.cu).
+// The merge behind the split-context attention cores (mla.cu, latent_attn.cu, grouped_attn.cu).
 #pragma once
 #include "common.cuh"
 
@@ -7,9 +7,12 @@ namespace blok {
 // ---------------------------------------------------------------------------
 // Merge of the split-KV partial results.  grid = (heads, B), 128 threads.
 //   part_o fp32 [B, splits, heads, kv_rank] unnormalised, part_ml fp32 [B, splits, heads, 2] = (max, sum)
+// Rows of o_lat are ldo values apart (0: heads * kv_rank).  gate, optional: bf16 [B, ld_gate]; head h's output times
+// sigmoid(gate[b][h]).
 // ---------------------------------------------------------------------------
 static __global__ void mla_merge_kernel(const float *__restrict__ part_o, const float *__restrict__ part_ml, int splits,
-                                 int heads, int kv_rank, uint16_t *__restrict__ o_lat) {
+                                 int heads, int kv_rank, uint16_t *__restrict__ o_lat, int ldo = 0,
+                                 const uint16_t *__restrict__ gate = nullptr, int ld_gate = 0) {
   extern __shared__ float s_wt[];  // [splits] weight of every split: exp(m_s - M), 0 for an empty split
   __shared__ float s_red[2][4];
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
@@ -31,7 +34,9 @@ static __global__ void mla_merge_kernel(const float *__restrict__ part_o, const 
   if ((tid & 31) == 0) s_red[1][tid >> 5] = L;
   __syncthreads();
   L = (s_red[1][0] + s_red[1][1]) + (s_red[1][2] + s_red[1][3]);
-  const float inv = L > 0.f ? 1.0f / L : 0.f;
+  float inv = L > 0.f ? 1.0f / L : 0.f;
+  if (gate) inv *= 1.0f / (1.0f + expf(-bf16_bits_to_f32(gate[(size_t)b * ld_gate + h])));
+  if (!ldo) ldo = heads * kv_rank;
   const float *po = part_o + ((size_t)b * splits * heads + h) * kv_rank;  // split s at + s * heads * kv_rank
   // four columns per thread, eight splits' worth of loads in flight per thread: the partial results (B x splits x 128 KB)
   // come from L2 or HBM, and the kernel is as fast as it keeps bytes in flight.  Each column still adds its splits in
@@ -65,7 +70,7 @@ static __global__ void mla_merge_kernel(const float *__restrict__ part_o, const 
     uint2 o;
     o.x = pack_bf16x2(acc.x * inv, acc.y * inv);
     o.y = pack_bf16x2(acc.z * inv, acc.w * inv);
-    *reinterpret_cast<uint2 *>(o_lat + ((size_t)b * heads + h) * kv_rank + (size_t)j4 * 4) = o;
+    *reinterpret_cast<uint2 *>(o_lat + (size_t)b * ldo + (size_t)h * kv_rank + (size_t)j4 * 4) = o;
   }
 }
 

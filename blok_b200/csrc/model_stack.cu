@@ -5,8 +5,8 @@
 // (a head's key size to 16, its value size to 16, everything a product contracts to 32), so that every activation is
 // aligned and the kernels need no bounds inside a head.  Padded values come out as zeros at every stage.
 //
-// A layer run is: streams + norm -> mixer -> streams + norm -> experts.  The streams' update by a sublayer's output is fused
-// with the norm in front of the next one (residual_streams.cu), across layer borders too.
+// A layer run is: residual + norm -> mixer -> residual + norm -> feed-forward.  The residual's update by a sublayer's output is
+// fused with the norm in front of the next one (residual_streams.cu, residual_norm.cu), across layer borders too.
 #include <algorithm>
 #include <cmath>
 #include <cstring>
@@ -16,6 +16,7 @@
 #include <utility>
 
 #include "gemm_tma.h"
+#include "prompt_attn_tc.h"
 #include "safetensors.h"
 #include "stack.h"
 #include "stack_kernels.h"
@@ -29,7 +30,7 @@ int launch_bf16_gemv_splitk(const uint16_t *w, const uint16_t *x, uint16_t *y_bf
                             cudaStream_t stream);
 int launch_head_gemv(const uint16_t *w, long w_head_stride, const uint16_t *x, long x_tok_stride, long x_head_stride, uint16_t *y, long y_tok_stride,
                      long y_head_stride, int rows, int cols, int heads, int T, cudaStream_t stream);
-int latent_prompt_take_error(unsigned *out);
+int launch_bf16_gateup(const uint16_t *gate, const uint16_t *up, const uint16_t *x, uint16_t *mid, int ffn, int cols, int T, cudaStream_t stream);
 int mla_attend_tc_take_error(unsigned *out);
 int launch_argmax_f32(const float *logits, int vocab, int pitch, int T, uint32_t *ids, cudaStream_t stream);
 
@@ -37,6 +38,7 @@ namespace {
 
 constexpr int kHeadRows = 64;       // rows of the vocabulary product per call
 constexpr int kShortPortion = 32;   // portions of up to this many tokens attend in the absorbed form
+constexpr int kSyntheticBuckets = 32; // distance buckets of a model without stored weights
 constexpr int kGemvAssignments = 64;  // up to this many (token, expert) pairs go through the mat-vec kernel
 
 int pad(int n, int to) { return (n + to - 1) / to * to; }
@@ -55,22 +57,29 @@ struct Hyper {
 struct LayerState {
   Norm norm1, norm2;
   Hyper hc1, hc2;
-  Mat qkvg, o;                       // linear
+  float *post1 = nullptr, *post2 = nullptr;  // sandwich: the norms behind the sublayers
+  Mat qkvg, o;                       // linear; state: everything that is projected in; grouped: q, k, v (unless borrowed), gates
   float *decay_pow = nullptr, *norm_w = nullptr;
   LinearAttn lin;                    // sizes only
   LatentShape lat;                   // latent
   Mat dqkv, uq, kvb;
   uint16_t *wuk_t = nullptr;         // [heads, rank, dim]
   float *q_norm = nullptr, *kv_norm = nullptr;
-  Mat up, down;                      // experts
+  StateInputs inputs;                // state: sizes and weights
+  int step_at = 0;                   // state: column of the step sizes
+  GroupedShape grp;                  // grouped
+  float *k_norm = nullptr;
+  int gate_at = 0;                   // grouped: column of the head gates
+  Mat up, down;                      // experts; dense: gate and up rows in `up`
   int *table = nullptr;
   ExpertPlan plan;
   int plan_index = -1;
 };
 struct Run {
   int layer = 0;
-  float *state = nullptr;  // linear: [slots, heads, dim, vdim]
-  void *pool = nullptr;    // latent: Act [pages, page_rows, row]
+  float *state = nullptr;  // linear, state: [slots, heads, dim, vdim]
+  void *pool = nullptr;    // latent, grouped: Act [pages, page_rows, row]; possibly an earlier run's
+  void *ring = nullptr;    // state: Act [slots, taps, channels]
 };
 
 struct StackModel {
@@ -79,13 +88,17 @@ struct StackModel {
   int W = 0, V = 0;  // padded width and vocabulary
   std::vector<LayerState> layers;
   std::vector<Run> runs;
-  uint16_t *embed = nullptr;
+  uint16_t *embed = nullptr, *bigram = nullptr;
+  double *turns = nullptr;       // sinusoid: turns per position of every pair of columns
+  uint32_t *last_ids = nullptr;  // [slots] newest token
   Norm final_norm;
   Mat head;
   ExpertPlanArgs *plans_dev = nullptr;
   int n_plans = 0, max_top = 1;
   // step buffers (Act: bf16 or fp32)
   float *x = nullptr, *y = nullptr, *ckr = nullptr, *lin_o = nullptr, *chunk_state = nullptr, *logits = nullptr;
+  float4 *token = nullptr;
+  void *xbc = nullptr;
   void *h = nullptr, *proj = nullptr, *cq = nullptr, *q_abs = nullptr, *o_lat = nullptr, *mix = nullptr, *mid = nullptr, *h_final = nullptr,
        *h_sel = nullptr;
   float *part_o = nullptr, *part_ml = nullptr;  // parts of split contexts
@@ -166,25 +179,36 @@ class Weights {
     if (int rc = gemm_operand_map(t->w, (long)rows, K, K, 128, &t->m128)) return rc;
     return gemm_operand_map(t->w, (long)rows, K, K, 256, &t->m256);
   }
-  // The stored matrix `name` into rows row0.. of t.
-  int fill(const Mat &t, long row0, const std::string &name, const Place &at, float std) {
-    return fill_rows(t.w + (size_t)row0 * t.K, t.K, name, at, std);
+  // The stored matrix `name` (or rows of it, see fill_rows) into rows row0.. of t.
+  int fill(const Mat &t, long row0, const std::string &name, const Place &at, float std, long from = 0, long total = 0) {
+    return fill_rows(t.w + (size_t)row0 * t.K, t.K, name, at, std, from, total);
   }
-  int fill_rows(uint16_t *dst, int ld, const std::string &name, const Place &at, float std) {
+  // Of a stored matrix of `total` rows, those from `from` on (total 0: all of it).
+  int fill_rows(uint16_t *dst, int ld, const std::string &name, const Place &at, float std, long from = 0, long total = 0) {
     if (!from_file_) {
       const size_t n = (size_t)at.rows * at.cols;
       fill_placed_kernel<<<(unsigned)((n + 255) / 256), 256>>>(dst, ld, at, next_key(), std);
       return launch_status("fill_placed_kernel");
     }
     const StoredTensor *t;
-    if (int rc = file_.need(name, "BF16", {at.rows, at.cols}, &t)) return rc;
+    if (int rc = file_.need(name, "BF16", {total ? total : at.rows, at.cols}, &t)) return rc;
     std::vector<uint16_t> raw((size_t)at.rows * at.cols);
-    if (int rc = file_.read(*t, raw.data())) return rc;
+    if (int rc = file_.read(*t, raw.data(), (uint64_t)from * at.cols * 2, raw.size() * 2)) return rc;
     const size_t prows = (size_t)at.row(at.rows - 1) + 1;
     std::vector<uint16_t> placed(prows * ld, 0);
     for (long r = 0; r < at.rows; ++r)
       for (int c = 0; c < at.cols; ++c) placed[(size_t)at.row(r) * ld + at.col(c)] = raw[(size_t)r * at.cols + c];
     BLOK_CUDA(cudaMemcpy(dst, placed.data(), placed.size() * 2, cudaMemcpyHostToDevice));
+    return BLOK_OK;
+  }
+  // Rows of a stored matrix of `cols` columns; `synthetic` without a file.
+  int stored_rows(const std::string &name, long cols, int synthetic, int *rows) {
+    *rows = synthetic;
+    if (!from_file_) return BLOK_OK;
+    const StoredTensor *t = file_.find(name);
+    BLOK_REQUIRE(t && t->shape.size() == 2 && t->shape[0] >= 1 && t->shape[0] < (1 << 20) && t->shape[1] == cols, BLOK_ERR_SHAPE,
+                 "tensor %s is missing or has not %ld columns", name.c_str(), cols);
+    *rows = (int)t->shape[0];
     return BLOK_OK;
   }
   int host_vector(const std::string &name, const std::vector<long> &shape, float mean, float dev, std::vector<float> *out) {
@@ -218,9 +242,10 @@ class Weights {
     for (int i = 0; i < n; ++i) p[i / group * gpad + i % group] = v[i];
     return upload(p, out);
   }
-  int norm(const std::string &name, int width, int padded, Norm *out) {
+  int norm(const std::string &name, int width, int padded, bool dynamic_tanh, Norm *out) {
     std::vector<float> a;
     int rc;
+    if (!dynamic_tanh) return vector(name, width, width, padded, padded, 1.f, 0.1f, &out->w);
     if ((rc = vector(name, width, width, padded, padded, 1.f, 0.1f, &out->w)) || (rc = vector(name + ".b", width, width, padded, padded, 0.f, 0.1f, &out->b)) ||
         (rc = host_vector(name + ".alpha", {}, 0.8f, 0.1f, &a)))
       return rc;
@@ -334,6 +359,133 @@ int load_latent(blok_model *m, Weights &w, const std::string &p, const LatentMix
   return w.fill(L.o, 0, p + "o", Place::in_heads(W, x.heads, x.vdim, s.vdim), fan(x.heads * x.vdim));
 }
 
+int load_state(blok_model *m, Weights &w, const std::string &p, const StateMixer &x, LayerState &L) {
+  StackModel *S = stack(m);
+  const int W = S->spec.width, dv = pad(x.vdim, 16), n = pad(x.state, 16);
+  const int inner = x.heads * x.vdim, hv = x.heads * dv, bc = x.groups * x.state, bcp = x.groups * n, channels = hv + 2 * bcp;
+  BLOK_REQUIRE(n <= kLinMaxDim, BLOK_ERR_SHAPE, "%s: a state of %d rows, at most %d are supported", p.c_str(), x.state, kLinMaxDim);
+  L.lin.heads = x.heads;
+  L.lin.dim = n;
+  L.lin.vdim = dv;
+  L.lin.share = x.heads / x.groups;
+  L.lin.v_first = true;
+  L.step_at = 2 * hv + 2 * bcp;
+  // z | x | B | C | steps
+  const long total = 2l * inner + 2 * bc + x.heads;
+  TRY(w.make(&L.qkvg, L.step_at + pad(x.heads, 16), S->W));
+  TRY(w.fill(L.qkvg, 0, p + "in", Place::out_heads(2 * x.heads, x.vdim, dv, W), fan(W), 0, total));
+  TRY(w.fill(L.qkvg, 2 * hv, p + "in", Place::out_heads(2 * x.groups, x.state, n, W), fan(W), 2l * inner, total));
+  TRY(w.fill(L.qkvg, L.step_at, p + "in", Place::plain(x.heads, W), fan(W), 2l * inner + 2 * bc, total));
+  TRY(w.make(&L.o, S->W, pad(hv, 32)));
+  TRY(w.fill(L.o, 0, p + "o", Place::in_heads(W, x.heads, x.vdim, dv), fan(inner)));
+  TRY(w.vector(p + "norm", inner, x.vdim, dv, hv, 1.f, 0.1f, &L.norm_w));
+  std::vector<float> conv, bias, placed_conv((size_t)x.taps * channels, 0.f), placed_bias((size_t)channels, 0.f);
+  TRY(w.host_vector(p + "conv", {inner + 2 * bc, x.taps}, 0.f, 1.f / std::sqrt((float)x.taps), &conv));
+  TRY(w.host_vector(p + "conv.b", {inner + 2 * bc}, 0.f, 0.1f, &bias));
+  for (int c = 0; c < inner + 2 * bc; ++c) {
+    const int at = c < inner ? c / x.vdim * dv + c % x.vdim : hv + (c - inner) / x.state * n + (c - inner) % x.state;
+    placed_bias[at] = bias[c];
+    for (int j = 0; j < x.taps; ++j) placed_conv[(size_t)j * channels + at] = conv[(size_t)c * x.taps + j];
+  }
+  float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *rate = nullptr, *skip = nullptr;
+  TRY(w.upload(placed_conv, &conv_w));
+  TRY(w.upload(placed_bias, &conv_b));
+  std::vector<float> a;
+  TRY(w.host_vector(p + "A_log", {x.heads}, 0.5f, 0.5f, &a));
+  for (float &v : a) v = (float)-std::exp((double)v);
+  TRY(w.upload(a, &rate));
+  TRY(w.vector(p + "dt_bias", x.heads, x.heads, x.heads, x.heads, -3.f, 1.f, &dt_bias));
+  TRY(w.vector(p + "D", x.heads, x.heads, x.heads, x.heads, 1.f, 0.2f, &skip));
+  L.lin.skip = skip;
+  StateInputs &s = L.inputs;
+  s.heads = x.heads;
+  s.channels = channels;
+  s.taps = x.taps;
+  s.conv_w = conv_w;
+  s.conv_b = conv_b;
+  s.dt_bias = dt_bias;
+  s.rate = rate;
+  s.ld = L.qkvg.R;
+  s.first = hv;
+  s.dt_at = L.step_at;
+  return BLOK_OK;
+}
+
+// The bucket of a distance: itself below half of them, then logarithmic up to `top`.
+int distance_bucket(int n, int buckets, double top) {
+  const int half = buckets / 2;
+  if (n < half) return n;
+  const double at = std::log((double)n / half) / std::log(top / half) * (buckets - half);
+  return std::min((double)(buckets - 1), half + std::floor(at));
+}
+
+int load_grouped(blok_model *m, Weights &w, const std::string &p, const GroupedMixer &x, LayerState &L) {
+  StackModel *S = stack(m);
+  const int W = S->spec.width;
+  GroupedShape &s = L.grp;
+  s.heads = x.heads;
+  s.kv_heads = x.kv_heads;
+  s.dim = pad(x.dim, 32);
+  s.vdim = pad(x.vdim, 16);
+  s.true_dim = x.dim;
+  s.scale = (float)x.scale;
+  s.eps = (float)S->spec.eps;
+  const bool own = x.kv_from < 0;
+  const int nq = x.heads * s.dim, nk = own ? x.kv_heads * s.dim : 0, nv = own ? x.kv_heads * s.vdim : 0;
+  L.gate_at = nq + nk + nv;
+  TRY(w.make(&L.qkvg, L.gate_at + (x.head_gate ? pad(x.heads, 16) : 0), S->W));
+  TRY(w.fill(L.qkvg, 0, p + "q", Place::out_heads(x.heads, x.dim, s.dim, W), fan(W)));
+  if (own) {
+    TRY(w.fill(L.qkvg, nq, p + "k", Place::out_heads(x.kv_heads, x.dim, s.dim, W), fan(W)));
+    TRY(w.fill(L.qkvg, nq + nk, p + "v", Place::out_heads(x.kv_heads, x.vdim, s.vdim, W), fan(W)));
+  }
+  if (x.head_gate) TRY(w.fill(L.qkvg, L.gate_at, p + "g", Place::plain(x.heads, W), fan(W)));
+  if (x.qk_norm) {
+    TRY(w.vector(p + "q.norm", x.heads * x.dim, x.dim, s.dim, nq, 1.f, 0.1f, &L.q_norm));
+    if (own) TRY(w.vector(p + "k.norm", x.kv_heads * x.dim, x.dim, s.dim, nk, 1.f, 0.1f, &L.k_norm));
+  }
+  if (x.bias_max > 0) {
+    int buckets = 0;
+    TRY(w.stored_rows(p + "rel", x.heads, kSyntheticBuckets, &buckets));
+    BLOK_REQUIRE(buckets >= 2 && x.bias_max > buckets / 2 && x.bias_max <= (1 << 24), BLOK_ERR_SHAPE, "%srel: %d buckets up to a distance of %g", p.c_str(),
+                 buckets, x.bias_max);
+    std::vector<float> rel, by_distance;
+    TRY(w.host_vector(p + "rel", {buckets, x.heads}, 0.f, 0.5f, &rel));
+    s.bias_len = 1;  // up to the first distance of the last bucket
+    while (distance_bucket(s.bias_len - 1, buckets, x.bias_max) < buckets - 1) ++s.bias_len;
+    by_distance.resize((size_t)x.heads * s.bias_len);
+    for (int n = 0; n < s.bias_len; ++n) {
+      const int b = distance_bucket(n, buckets, x.bias_max);
+      for (int h = 0; h < x.heads; ++h) by_distance[(size_t)h * s.bias_len + n] = rel[(size_t)b * x.heads + h];
+    }
+    float *bias = nullptr;
+    TRY(w.upload(by_distance, &bias));
+    s.bias = bias;
+  }
+  TRY(w.make(&L.o, S->W, pad(x.heads * s.vdim, 32)));
+  return w.fill(L.o, 0, p + "o", Place::in_heads(W, x.heads, x.vdim, s.vdim), fan(x.heads * x.vdim));
+}
+
+int load_mixer(blok_model *m, Weights &w, const std::string &p, const StackLayer &x, LayerState &L) {
+  switch (x.kind) {
+    case StackLayer::Linear: return load_linear(m, w, p, x.linear, L);
+    case StackLayer::Latent: return load_latent(m, w, p, x.latent, L);
+    case StackLayer::State: return load_state(m, w, p, x.state, L);
+    case StackLayer::Grouped: return load_grouped(m, w, p, x.grouped, L);
+  }
+  return BLOK_ERR_STATE;
+}
+
+int load_dense(blok_model *m, Weights &w, const std::string &p, const DenseGated &x, LayerState &L) {
+  StackModel *S = stack(m);
+  const int W = S->spec.width, ff = pad(x.ff, 32);
+  TRY(w.make(&L.up, 2 * ff, S->W));
+  TRY(w.fill(L.up, 0, p + "gate", Place::plain(x.ff, W), fan(W)));
+  TRY(w.fill(L.up, ff, p + "up", Place::plain(x.ff, W), fan(W)));
+  TRY(w.make(&L.down, S->W, ff));
+  return w.fill(L.down, 0, p + "down", Place::plain(W, x.ff), fan(x.ff));
+}
+
 int load_experts(blok_model *m, Weights &w, const std::string &p, const TableExperts &x, LayerState &L) {
   StackModel *S = stack(m);
   const int W = S->spec.width, ff = pad(x.ff, 32);
@@ -414,6 +566,10 @@ int product(StackModel *S, const Mat &w, const void *x, int T, void *y, bool y_f
 }  // namespace
 
 int stack_describe(blok_model *m, const StackSpec &spec) {
+  BLOK_REQUIRE(spec.sandwich ? spec.streams == 1 : spec.embed_scale == 1 && !spec.bigram_buckets && !spec.sinusoid && spec.logit_scale == 1, BLOK_ERR_ARG,
+               "this form of the residual does not go with the other values");
+  for (const StackLayer &L : spec.layers)
+    BLOK_REQUIRE(!spec.sandwich || L.ff_kind != StackLayer::Experts, BLOK_ERR_ARG, "experts do not go with sandwiched sublayers");
   BLOK_REQUIRE(spec.streams <= kMaxStreams && !spec.order.empty(), BLOK_ERR_SHAPE, "%d residual streams (at most %d), %zu layer runs", spec.streams,
                kMaxStreams, spec.order.size());
   StackModel *S = new (std::nothrow) StackModel();
@@ -445,7 +601,27 @@ int stack_build(blok_model *m, const char *dir, uint64_t seed) {
   TRY(w.zeroed((size_t)spec.vocab * S->W * 2, &p));
   S->embed = static_cast<uint16_t *>(p);
   TRY(w.fill_rows(S->embed, S->W, "embed", Place::plain(spec.vocab, spec.width), 1.0f));
-  TRY(w.norm("final.norm", spec.width, S->W, &S->final_norm));
+  if (spec.bigram_buckets) {
+    TRY(w.zeroed(((size_t)spec.bigram_buckets + 1) * S->W * 2, &p));
+    S->bigram = static_cast<uint16_t *>(p);
+    TRY(w.fill_rows(S->bigram, S->W, "bigram", Place::plain(spec.bigram_buckets + 1, spec.width), 1.0f));
+    TRY(w.zeroed((size_t)c.max_batch * 4, &p));
+    S->last_ids = static_cast<uint32_t *>(p);
+  }
+  if (spec.sinusoid) {
+    std::vector<double> turns((size_t)S->W / 2);
+    for (int i = 0; i < S->W / 2; ++i) turns[i] = std::pow(10000.0, -2.0 * i / spec.width) / 6.28318530717958647693;
+    TRY(dev_alloc_as(m, turns.size(), &S->turns));
+    BLOK_CUDA(cudaMemcpy(S->turns, turns.data(), turns.size() * sizeof(double), cudaMemcpyHostToDevice));
+  }
+  if (spec.sandwich) {  // the logits' scale rides on the last norm
+    std::vector<float> f, padded((size_t)S->W, 0.f);
+    TRY(w.host_vector("final.norm", {spec.width}, 1.f, 0.1f, &f));
+    for (int i = 0; i < spec.width; ++i) padded[i] = (float)(f[i] * spec.logit_scale);
+    TRY(w.upload(padded, &S->final_norm.w));
+  } else {
+    TRY(w.norm("final.norm", spec.width, S->W, true, &S->final_norm));
+  }
   TRY(w.make(&S->head, S->V, S->W));
   TRY(w.fill(S->head, 0, "head", Place::plain(spec.vocab, spec.width), fan(spec.width)));
   S->layers.resize(spec.layers.size());
@@ -453,30 +629,50 @@ int stack_build(blok_model *m, const char *dir, uint64_t seed) {
     const StackLayer &x = spec.layers[i];
     LayerState &L = S->layers[i];
     const std::string pl = "l" + std::to_string(i) + ".";
-    TRY(w.norm(pl + "norm1", spec.width, S->W, &L.norm1));
-    TRY(w.hyper(pl + "hc1", spec.streams, &L.hc1));
-    TRY(x.kind == StackLayer::Linear ? load_linear(m, w, pl + "mix.", x.linear, L) : load_latent(m, w, pl + "mix.", x.latent, L));
-    if (x.has_ff) {
-      TRY(w.norm(pl + "norm2", spec.width, S->W, &L.norm2));
-      TRY(w.hyper(pl + "hc2", spec.streams, &L.hc2));
-      TRY(load_experts(m, w, pl + "mlp.", x.ff, L));
-      S->max_top = std::max(S->max_top, x.ff.top);
+    TRY(w.norm(pl + "norm1", spec.width, S->W, !spec.sandwich, &L.norm1));
+    if (spec.sandwich) TRY(w.vector(pl + "norm1b", spec.width, spec.width, S->W, S->W, 1.f, 0.1f, &L.post1));
+    else TRY(w.hyper(pl + "hc1", spec.streams, &L.hc1));
+    TRY(load_mixer(m, w, pl + "mix.", x, L));
+    if (x.ff_kind != StackLayer::NoFf) {
+      TRY(w.norm(pl + "norm2", spec.width, S->W, !spec.sandwich, &L.norm2));
+      if (spec.sandwich) TRY(w.vector(pl + "norm2b", spec.width, spec.width, S->W, S->W, 1.f, 0.1f, &L.post2));
+      else TRY(w.hyper(pl + "hc2", spec.streams, &L.hc2));
+      TRY(x.ff_kind == StackLayer::Dense ? load_dense(m, w, pl + "mlp.", x.dense, L) : load_experts(m, w, pl + "mlp.", x.ff, L));
+      if (x.ff_kind == StackLayer::Experts) S->max_top = std::max(S->max_top, x.ff.top);
     }
   }
 
   // caches and states: one per run
   const size_t esz = S->f32 ? 4 : 2, N = (size_t)m->rows;
+  std::vector<void *> pool_of(spec.layers.size(), nullptr);
   for (int l : spec.order) {
     Run r;
     r.layer = l;
+    const StackLayer &x = spec.layers[l];
     const LayerState &L = S->layers[l];
-    if (spec.layers[l].kind == StackLayer::Linear) TRY(dev_alloc_as(m, (size_t)c.max_batch * L.lin.heads * L.lin.dim * L.lin.vdim, &r.state));
-    else TRY(dev_alloc(m, (size_t)c.kv_pages * c.kv_page_rows * L.lat.row() * esz, &r.pool));
+    const size_t rows = (size_t)c.kv_pages * c.kv_page_rows;
+    switch (x.kind) {
+      case StackLayer::State:
+        TRY(w.zeroed((size_t)c.max_batch * L.inputs.taps * L.inputs.channels * esz, &r.ring));
+        // fall through
+      case StackLayer::Linear:
+        TRY(dev_alloc_as(m, (size_t)c.max_batch * L.lin.heads * L.lin.dim * L.lin.vdim, &r.state));
+        break;
+      case StackLayer::Latent:
+        TRY(dev_alloc(m, rows * L.lat.row() * esz, &r.pool));
+        break;
+      case StackLayer::Grouped:  // finite from the start: whole boxes are copied from it
+        if (x.grouped.kv_from >= 0) r.pool = pool_of[x.grouped.kv_from];
+        else TRY(w.zeroed(rows * L.grp.row() * esz, &r.pool));
+        BLOK_REQUIRE(r.pool, BLOK_ERR_STATE, "layer %d has no keys to borrow", l);
+        break;
+    }
+    pool_of[l] = r.pool;
     S->runs.push_back(r);
   }
 
   // step buffers, sized for the largest layer
-  size_t proj = 1, ckr = 1, cq = 1, q_abs = 1, o_lat = 1, lin_o = 1, mixw = 1, mid = 1, chunk_state = 1, part_o = 1, part_ml = 1, c_all = 1, kr_all = 1, kv_all = 1;
+  size_t proj = 1, ckr = 1, cq = 1, q_abs = 1, o_lat = 1, lin_o = 1, mixw = 1, mid = 1, chunk_state = 1, part_o = 1, part_ml = 1, c_all = 1, kr_all = 1, kv_all = 1, xbc = 1, token = 1;
   int max_R = S->V;
   std::vector<const Mat *> mats = {&S->head};
   for (size_t i = 0; i < spec.layers.size(); ++i) {
@@ -484,9 +680,21 @@ int stack_build(blok_model *m, const char *dir, uint64_t seed) {
     const LayerState &L = S->layers[i];
     mats.push_back(&L.o);
     mixw = std::max(mixw, (size_t)L.o.K);
-    if (x.kind == StackLayer::Linear) {
+    if (x.kind == StackLayer::Grouped) {
+      const GroupedShape &s = L.grp;
       mats.push_back(&L.qkvg);
       proj = std::max(proj, (size_t)L.qkvg.R);
+      const int short_rows = !S->f32 && grouped_prompt_supports(s) ? std::min(m->rows, std::max(c.max_batch, kShortPortion)) : m->rows;
+      const size_t parts = S->f32 ? 0 : grouped_attend_max_parts(s, short_rows, c.max_ctx);
+      part_o = std::max(part_o, parts * s.heads * s.vdim);
+      part_ml = std::max(part_ml, parts * s.heads * 2);
+    } else if (x.kind == StackLayer::Linear || x.kind == StackLayer::State) {
+      mats.push_back(&L.qkvg);
+      proj = std::max(proj, (size_t)L.qkvg.R);
+      if (x.kind == StackLayer::State) {
+        xbc = std::max(xbc, (size_t)L.inputs.channels);
+        token = std::max(token, (size_t)L.inputs.heads);
+      }
       lin_o = std::max(lin_o, (size_t)L.lin.heads * L.lin.vdim);
       if (!S->f32) chunk_state = std::max(chunk_state, linear_chunk_scratch_bytes(L.lin.heads, L.lin.dim, L.lin.vdim, c.prefill_chunk));
     } else {
@@ -510,7 +718,13 @@ int stack_build(blok_model *m, const char *dir, uint64_t seed) {
         kv_all = std::max(kv_all, ctx * L.kvb.R);
       }
     }
-    if (x.has_ff) mid = std::max(mid, (size_t)x.ff.top * pad(x.ff.ff, 32));
+    if (x.ff_kind == StackLayer::Experts) mid = std::max(mid, (size_t)x.ff.top * pad(x.ff.ff, 32));
+    if (x.ff_kind == StackLayer::Dense) {
+      mats.push_back(&L.down);
+      mid = std::max(mid, (size_t)L.down.K);
+      if (S->f32) proj = std::max(proj, (size_t)L.up.R);
+      S->splitk_bytes = std::max(S->splitk_bytes, wgemm_splitk_bytes(WG_BF16_SWIGLU, L.up.K, L.down.K, kWgStreamTokens));
+    }
   }
   for (const Mat *t : mats) {
     max_R = std::max(max_R, t->R);
@@ -528,6 +742,8 @@ int stack_build(blok_model *m, const char *dir, uint64_t seed) {
   TRY(buffer(m, part_o * 4, &S->part_o));
   TRY(buffer(m, part_ml * 4, &S->part_ml));
   TRY(buffer(m, N * lin_o * 4, &S->lin_o));
+  TRY(buffer(m, N * xbc * esz, &S->xbc));
+  TRY(buffer(m, N * token * sizeof(float4), &S->token));
   TRY(buffer(m, chunk_state, &S->chunk_state));
   TRY(buffer(m, (N + slack) * mixw * esz, &S->mix));
   TRY(buffer(m, (N + slack) * mid * esz, &S->mid));
@@ -545,7 +761,7 @@ int stack_build(blok_model *m, const char *dir, uint64_t seed) {
   // expert plans, one per layer
   std::vector<ExpertPlanArgs> plans;
   for (size_t i = 0; i < spec.layers.size(); ++i) {
-    if (!spec.layers[i].has_ff || S->f32) continue;
+    if (spec.layers[i].ff_kind != StackLayer::Experts || S->f32) continue;
     LayerState &L = S->layers[i];
     const TableExperts &x = spec.layers[i].ff;
     const int tiles = expert_plan_max_tiles(m->rows * x.top, x.experts);
@@ -674,6 +890,113 @@ int run_latent(const Call &c, const LayerState &L, const Run &r) {
   return product(S, L.o, S->mix, c.T, S->y, true, c.stream);
 }
 
+// S->h -> S->y: a selective state space.
+int run_state(const Call &c, const StateMixer &x, const LayerState &L, const Run &r) {
+  StackModel *S = c.S;
+  TRY(product(S, L.qkvg, S->h, c.T, S->proj, false, c.stream));
+  StateInputs in = L.inputs;
+  in.proj = S->proj;
+  in.f32 = S->f32;
+  in.ring = r.ring;
+  in.out = S->xbc;
+  in.token = S->token;
+  in.token_ld = c.m->rows;
+  TRY(launch_state_inputs(in, c.rows, c.T, c.chunk, c.stream));
+  LinearAttn a = L.lin;
+  a.qkvg = S->xbc;
+  a.ld = in.channels;
+  a.f32 = S->f32;
+  a.token = S->token;
+  a.token_ld = in.token_ld;
+  a.state = r.state;
+  a.o = S->lin_o;
+  a.chunk_state = S->chunk_state;
+  if (c.chunk) TRY(launch_linear_chunk(a, c.m->chunk_slot, c.m->host_pos[c.m->chunk_slot], c.T, c.stream));
+  else TRY(launch_linear_step(a, c.rows, c.T, c.stream));
+  GatedNorm g;
+  g.heads = x.heads;
+  g.vdim = L.lin.vdim;
+  g.true_vdim = x.vdim;
+  g.w = L.norm_w;
+  g.eps = (float)S->spec.eps;
+  g.o = S->lin_o;
+  g.g = S->proj;
+  g.ldg = L.qkvg.R;
+  g.out = S->mix;
+  g.ldo = L.o.K;
+  g.f32 = S->f32;
+  TRY(launch_gate_then_norm(g, x.norm_groups, c.T, c.stream));
+  return product(S, L.o, S->mix, c.T, S->y, true, c.stream);
+}
+
+template <typename Act>
+GroupedQuery<Act> grouped_query(const StackModel *S, const GroupedMixer &x, const LayerState &L) {
+  GroupedQuery<Act> q;
+  q.q = static_cast<const Act *>(S->proj);
+  q.ldq = L.qkvg.R;
+  if (x.head_gate) q.gate = q.q + L.gate_at;
+  q.ld_gate = L.qkvg.R;
+  q.out = static_cast<Act *>(S->mix);
+  q.ldo = L.o.K;
+  return q;
+}
+
+// S->h -> S->y: grouped attention.
+int run_grouped(const Call &c, const GroupedMixer &x, const LayerState &L, const Run &r) {
+  StackModel *S = c.S;
+  const GroupedShape &s = L.grp;
+  TRY(product(S, L.qkvg, S->h, c.T, S->proj, false, c.stream));
+  if (x.qk_norm || x.kv_from < 0)
+    TRY(launch_grouped_append(s, S->proj, L.qkvg.R, L.q_norm, L.k_norm, c.rows, c.T, x.kv_from < 0 ? r.pool : nullptr, S->f32, c.stream));
+  if (S->f32) {
+    TRY(launch_grouped_attend_f32(s, grouped_query<float>(S, x, L), r.pool, c.rows, c.T, c.stream));
+  } else if (c.chunk && c.T > kShortPortion && grouped_prompt_supports(s)) {
+    const int slot = c.m->chunk_slot, n = (int)c.m->host_pos[slot] + c.T;
+    const long rows = (long)c.m->cfg.kv_pages * c.m->cfg.kv_page_rows;
+    TRY(launch_grouped_prompt(s, grouped_query<uint16_t>(S, x, L), r.pool, rows, c.rows, slot, c.T, n, c.stream));
+  } else {
+    TRY(launch_grouped_attend(s, grouped_query<uint16_t>(S, x, L), r.pool, c.rows, c.T, c.m->cfg.max_ctx, S->part_o, S->part_ml, c.stream));
+  }
+  return product(S, L.o, S->mix, c.T, S->y, true, c.stream);
+}
+
+int run_mixer(const Call &c, const StackLayer &x, const LayerState &L, const Run &r) {
+  switch (x.kind) {
+    case StackLayer::Linear: return run_linear(c, x.linear, L, r);
+    case StackLayer::Latent: return run_latent(c, L, r);
+    case StackLayer::State: return run_state(c, x.state, L, r);
+    case StackLayer::Grouped: return run_grouped(c, x.grouped, L, r);
+  }
+  return BLOK_ERR_STATE;
+}
+
+// S->h -> S->y: the gated feed-forward.
+int run_dense(const Call &c, const LayerState &L) {
+  StackModel *S = c.S;
+  const int ff = L.down.K;
+  const uint16_t *h = static_cast<const uint16_t *>(S->h), *up = L.up.w + (size_t)ff * L.up.K;
+  uint16_t *mid = static_cast<uint16_t *>(S->mid);
+  if (S->f32) {
+    TRY(product(S, L.up, S->h, c.T, S->proj, false, c.stream));
+    TRY(launch_swiglu_f32(static_cast<const float *>(S->proj), static_cast<float *>(S->mid), ff, c.T, c.stream));
+  } else if (c.T <= 8 && ((size_t)L.up.K * 2 + 64) * c.T <= 200 * 1024) {
+    TRY(launch_bf16_gateup(L.up.w, up, h, mid, ff, L.up.K, c.T, c.stream));
+  } else if (c.T > 8 && c.T <= kWgStreamTokens && L.up.K % 256 == 0) {
+    TRY(launch_wgemm_rows(WG_BF16_SWIGLU, L.up.w, up, h, mid, nullptr, ff, L.up.K, c.T, S->splitk_ws, S->splitk_bytes, c.stream));
+  } else {
+    GemmTma g;
+    TRY(x_map(S, S->h, L.up.K, &g.x));
+    g.w128 = &L.up.m128;
+    g.T = c.T;
+    g.R = g.ldo = g.up_row = ff;
+    g.K = L.up.K;
+    g.act = GEMM_ACT_SWIGLU;
+    g.out = mid;
+    TRY(launch_gemm_tma(g, c.stream));
+  }
+  return product(S, L.down, S->mid, c.T, S->y, true, c.stream);
+}
+
 bool planned(const StackModel *S, int T, int top) { return !S->f32 && T * top > kGemvAssignments; }
 
 // S->h (in expert order when planned) -> S->y, one row per assignment.
@@ -710,6 +1033,60 @@ int run_experts(const Call &c, const TableExperts &x, const LayerState &L) {
   return launch_gemm_tma(g, c.stream);
 }
 
+// The layers around one residual with a norm on both sides of every sublayer.
+int sandwich_layers(const Call &c) {
+  blok_model *m = c.m;
+  StackModel *S = c.S;
+  const StackSpec &spec = S->spec;
+  ResidualNorm a;
+  a.T = c.T;
+  a.width = S->W;
+  a.true_width = spec.width;
+  a.x = S->x;
+  a.embed = S->embed;
+  a.vocab = spec.vocab;
+  a.embed_scale = (float)spec.embed_scale;
+  a.bigram = S->bigram;
+  a.buckets = spec.bigram_buckets;
+  a.mul_prev = spec.bigram_mul_prev;
+  a.mul_cur = spec.bigram_mul_cur;
+  a.turns = S->turns;
+  a.last_ids = S->last_ids;
+  a.pos = c.rows.pos;
+  a.slot_of = c.rows.slot_of;
+  a.chunk = c.chunk;
+  a.mult = (float)spec.residual_mult;
+  a.eps = (float)spec.eps;
+  a.h = S->h;
+  a.h_f32 = S->f32;
+  a.ids = m->ids;
+  auto step = [&](const Norm &n) {
+    a.norm_w = n.w;
+    const int rc = launch_residual_norm(a, c.stream);
+    a.ids = nullptr;
+    a.copy = nullptr;
+    a.y = S->y;
+    return rc;
+  };
+  for (size_t i = 0; i < S->runs.size(); ++i) {
+    const Run &r = S->runs[i];
+    const StackLayer &x = spec.layers[r.layer];
+    const LayerState &L = S->layers[r.layer];
+    TRY(step(L.norm1));
+    TRY(run_mixer(c, x, L, r));
+    a.post_w = L.post1;
+    if (x.ff_kind == StackLayer::Dense) {
+      TRY(step(L.norm2));
+      TRY(run_dense(c, L));
+      a.post_w = L.post2;
+    }
+    if (m->trace && c.T <= m->trace_rows) a.copy = m->trace + i * (size_t)m->trace_rows * spec.width;
+  }
+  a.h = S->h_final;
+  if (S->last_ids) a.keep_ids = m->ids;
+  return step(S->final_norm);
+}
+
 }  // namespace
 
 int stack_layers(blok_model *m, int T, bool chunk, blok_stream_t stream_) {
@@ -726,9 +1103,10 @@ int stack_layers(blok_model *m, int T, bool chunk, blok_stream_t stream_) {
   c.rows.table = m->table_dev;
   c.rows.table_stride = m->table_stride;
   c.rows.page_rows = m->cfg.kv_page_rows;
+  if (spec.sandwich) return sandwich_layers(c);
   if (S->n_plans) {
     bool any = false;
-    for (const StackLayer &L : spec.layers) any = any || (L.has_ff && planned(S, T, L.ff.top));
+    for (const StackLayer &L : spec.layers) any = any || (L.ff_kind == StackLayer::Experts && planned(S, T, L.ff.top));
     if (any) TRY(launch_expert_plan(S->plans_dev, S->n_plans, m->ids, spec.vocab, T, c.stream));
   }
   // what the streams have still to take in
@@ -768,9 +1146,9 @@ int stack_layers(blok_model *m, int T, bool chunk, blok_stream_t stream_) {
     const StackLayer &x = spec.layers[r.layer];
     const LayerState &L = S->layers[r.layer];
     TRY(step(L.hc1.in, L.norm1));
-    TRY(x.kind == StackLayer::Linear ? run_linear(c, x.linear, L, r) : run_latent(c, L, r));
+    TRY(run_mixer(c, x, L, r));
     took(L.hc1, 1, nullptr);
-    if (x.has_ff) {
+    if (x.ff_kind == StackLayer::Experts) {
       const bool plan = planned(S, T, x.ff.top);
       if (plan) {
         a.copies = x.ff.top;
@@ -779,6 +1157,10 @@ int stack_layers(blok_model *m, int T, bool chunk, blok_stream_t stream_) {
       TRY(step(L.hc2.in, L.norm2));
       TRY(run_experts(c, x.ff, L));
       took(L.hc2, x.ff.top, plan ? L.plan.at : nullptr);
+    } else if (x.ff_kind == StackLayer::Dense) {
+      TRY(step(L.hc2.in, L.norm2));
+      TRY(run_dense(c, L));
+      took(L.hc2, 1, nullptr);
     }
     if (m->trace && T <= m->trace_rows) a.sum = m->trace + i * (size_t)m->trace_rows * spec.width;
   }
@@ -822,8 +1204,8 @@ int stack_check(blok_model *, blok_stream_t stream) {
   unsigned err = 0;
   TRY(gemm_tma_take_error(&err));
   BLOK_REQUIRE(!err, BLOK_ERR_TIMEOUT, "a product gave up on a barrier");
-  TRY(latent_prompt_take_error(&err));
-  BLOK_REQUIRE(!err, BLOK_ERR_TIMEOUT, "latent attention over a prompt gave up on a barrier");
+  TRY(prompt_attn_take_error(&err));
+  BLOK_REQUIRE(!err, BLOK_ERR_TIMEOUT, "attention over a prompt gave up on a barrier");
   TRY(mla_attend_tc_take_error(&err));
   BLOK_REQUIRE(!err, BLOK_ERR_TIMEOUT, "the attention core gave up on wait %u", err);
   return BLOK_OK;

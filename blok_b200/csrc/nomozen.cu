@@ -7,72 +7,12 @@
 //   loop            layers start .. stop - 1 run `times` times in a row with the same weights and caches of their own
 #include <cmath>
 
+#include "config_fields.h"
 #include "stack.h"
 #include "stack_kernels.h"
 
 namespace blok {
 namespace {
-
-// Reads fields of one JSON object; the first field that is missing or of another kind leaves an error.
-class Fields {
- public:
-  Fields(const Json *object, std::string where) : j_(object), where_(std::move(where)) {
-    if (!j_ || j_->kind != Json::Object) fail("is not an object");
-  }
-  int rc() const { return rc_; }
-  double number(const char *name) {
-    const Json *v = get(name);
-    if (v && v->kind != Json::Number) fail(name, "is not a number");
-    return v && v->kind == Json::Number ? v->number : 0;
-  }
-  int size(const char *name) {
-    const double v = number(name);
-    if (!rc_ && !(v >= 1 && v <= (1 << 30) && v == std::floor(v))) fail(name, "is not a positive integer");
-    return rc_ ? 0 : (int)v;
-  }
-  std::string text(const char *name) {
-    const Json *v = get(name);
-    if (v && v->kind != Json::String) fail(name, "is not a string");
-    return v ? v->text : std::string();
-  }
-  std::vector<double> numbers(const char *name) {
-    std::vector<double> out;
-    const Json *v = get(name);
-    if (v && v->kind != Json::Array) fail(name, "is not a list");
-    if (v)
-      for (const Json &x : v->items) {
-        if (x.kind != Json::Number) fail(name, "holds something else than numbers");
-        out.push_back(x.number);
-      }
-    return out;
-  }
-  // A field that is an object; after an error here its fields report nothing more.
-  Fields object(const char *name) {
-    const Json *v = get(name);
-    if (!rc_) return Fields(v, where_ + "." + name);
-    Fields none;
-    none.rc_ = rc_;
-    return none;
-  }
-  void fail(const char *name, const char *what) { fail((std::string(name) + " " + what).c_str()); }
-
- private:
-  const Json *j_ = nullptr;
-  std::string where_;
-  int rc_ = BLOK_OK;
-
-  Fields() = default;
-  const Json *get(const char *name) {
-    if (rc_) return nullptr;
-    const Json *v = j_->find(name);
-    if (!v) fail(name, "is missing");
-    return v;
-  }
-  void fail(const char *what) {
-    if (!rc_) set_error("config.json: %s: %s", where_.c_str(), what);
-    rc_ = BLOK_ERR_ARG;
-  }
-};
 
 int read_linear(const Json *mixer, const std::string &where, bool lightning, LinearMixer *out) {
   Fields f(mixer, where);
@@ -142,7 +82,7 @@ int configure(blok_model *m, const Json &config) {
       Fields ff(mlp, where + ".mlp");
       const std::string kind = ff.text("kind");
       Fields router = ff.object("router"), expert = ff.object("expert");
-      L.has_ff = true;
+      L.ff_kind = StackLayer::Experts;
       L.ff.experts = router.size("experts");
       L.ff.top = router.size("top");
       L.ff.ff = expert.size("ff");

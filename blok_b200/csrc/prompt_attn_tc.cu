@@ -1,10 +1,13 @@
-// The prompt form of latent attention (latent_attn.cu) on tcgen05: causal attention of T queries over n per-head keys and
-// values, for a query-key size of 128 to 256 and a value size of 64 or 128, in multiples of 64.
+// Softmax attention of a prompt on tcgen05: causal attention of T queries over n keys and values, for the prompt form of latent
+// attention (per-head keys and values, latent_attn.cu) and for grouped attention over cached pages (grouped_attn.cu).  Query-key
+// sizes up to 256 and value sizes up to 128.
 //
 // A CTA owns 128 queries of one head and walks the keys in tiles of 64:
 //   S [queries x 64]   = Q K^T    both operands in shared memory (TMA, 128-byte swizzle), accumulator in tensor memory, two
 //                                 buffers
-//   P = exp2(S * scale * log2 e - m)   one query per thread: no exchange between threads for its maximum and sum
+//   P = exp2(S * scale * log2 e + bias - m)   one query per thread: no exchange between threads for its maximum and sum.  A bias
+//                                 depends on the distance alone: a warp's 32 queries meet 64 keys at 95 distances, which the
+//                                 warp puts into shared memory with the causal mask in them
 //   O [queries x vdim] += P V     P in tensor memory as the A operand, in three bf16 parts (bf16_split.cuh); V is read from
 //                                 its rows as they are (MN-major B operand)
 // The scores of tile n + 1 are computed under the softmax of tile n.  The running maximum is kept lazily: a row's reference
@@ -16,6 +19,7 @@
 
 #include "bf16_split.cuh"
 #include "gemm_tma.h"
+#include "prompt_attn_tc.h"
 #include "stack_kernels.h"
 #include "tc_pipe.cuh"
 
@@ -26,9 +30,10 @@ constexpr int kPtQChunk = kPtRows * 128, kPtKChunk = kPtKeys * 128;  // bytes of
 constexpr int kPtMaxQ = 4;                                           // chunks of a query
 constexpr int kPtColS = 0, kPtColP = 128, kPtColO = 384;             // tensor memory: S 2 x 64, P 2 x 3 x 32 (of 4 x 64), O
 constexpr int kPtTmemCols = 512;
+constexpr float kPtLog2e = 1.4426950408889634f;
 constexpr float kPtLazy = 57.7f;  // 40 natural units in the log2 domain
 
-__device__ unsigned g_latent_prompt_error = 0;
+__device__ unsigned g_prompt_attn_error = 0;
 
 __device__ __forceinline__ float pt_ex2(float x) {
   float y;
@@ -36,23 +41,20 @@ __device__ __forceinline__ float pt_ex2(float x) {
   return y;
 }
 
-struct PtArgs {
-  uint16_t *out;
-  int T, n, ldo, heads, dim, rot, vdim;
-  float scale_log2;
-};
-
+// BIAS: scores take a bias by distance.
+template <bool BIAS>
 __global__ void __launch_bounds__(kPtThreads, 1)
-    latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mkv, const __grid_constant__ CUtensorMap mkr,
-                            const PtArgs a) {
+    prompt_attn_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mkv, const __grid_constant__ CUtensorMap mkr,
+                          const PromptAttn a) {
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(8) unsigned long long s_bar[2 * kPtStages + 9];
   __shared__ uint32_t s_tmem;
+  __shared__ float s_window[BIAS ? 4 : 1][BIAS ? 96 : 1];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h = blockIdx.y, q0 = (gridDim.x - 1 - blockIdx.x) * kPtRows;  // the longest rows of tiles start first
   const int first = a.n - a.T, nq = min(kPtRows, a.T - q0);
   const int nt = (first + q0 + nq + kPtKeys - 1) / kPtKeys;
-  const int qc = (a.dim + a.rot) / 64, dc = a.dim / 64, vc = a.vdim / 64;
+  const int qc = (a.dim + 63) / 64, vc = (a.vdim + 63) / 64, kh = h / a.share;
   const uint32_t sQ = ((uint32_t)__cvta_generic_to_shared(smem_raw) + 1023u) & ~1023u;
   const uint32_t stage_bytes = (uint32_t)(qc + vc) * kPtKChunk, sT = sQ + (uint32_t)qc * kPtQChunk;
   const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&s_bar[0]);
@@ -82,19 +84,30 @@ __global__ void __launch_bounds__(kPtThreads, 1)
   if (warp == 4) {
     if (lane == 0) {
       tp_expect_tx(qfull, (uint32_t)qc * kPtQChunk);
-      for (int c = 0; c < qc; ++c) tp_load_2d(sQ + c * kPtQChunk, &mq, h * (a.dim + a.rot) + 64 * c, q0, qfull);
+      for (int c = 0; c < qc; ++c) tp_load_2d(sQ + c * kPtQChunk, &mq, h * a.q_head + 64 * c, q0, qfull);
+      // the row of key j: its page's, or j itself.  A box past the last key repeats the tile's first; its keys take no weight.
+      auto row_of = [&](int j) { return a.table ? a.table[j / a.page_rows] * a.page_rows + j % a.page_rows : j; };
+      int next[2] = {row_of(0), a.box < kPtKeys ? row_of(a.box < a.n ? a.box : 0) : 0};
       int issued = 0;
       for (int n = 0; n < nt; ++n) {
-        const int s = n % kPtStages;
+        const int s = n % kPtStages, row[2] = {next[0], next[1]};
+        if (n + 1 < nt) {
+          const int j = (n + 1) * kPtKeys;
+          next[0] = row_of(j);
+          if (a.box < kPtKeys) next[1] = row_of(j + a.box < a.n ? j + a.box : j);
+        }
         if (n >= kPtStages && !tp_wait(empty + 8 * s, (uint32_t)((n / kPtStages - 1) & 1))) {
           failed = true;
           break;
         }
         const uint32_t dst = sT + (uint32_t)s * stage_bytes, f = full + 8 * s;
         tp_expect_tx(f, stage_bytes);
-        for (int c = 0; c < dc; ++c) tp_load_2d(dst + c * kPtKChunk, &mkv, h * a.dim + 64 * c, n * kPtKeys, f);
-        for (int c = dc; c < qc; ++c) tp_load_2d(dst + c * kPtKChunk, &mkr, 64 * (c - dc), n * kPtKeys, f);
-        for (int c = 0; c < vc; ++c) tp_load_2d(dst + (qc + c) * kPtKChunk, &mkv, a.heads * a.dim + h * a.vdim + 64 * c, n * kPtKeys, f);
+        for (int p = 0; p * a.box < kPtKeys; ++p) {
+          const uint32_t to = dst + p * a.box * 128;
+          for (int c = 0; c < a.key_chunks; ++c) tp_load_2d(to + c * kPtKChunk, &mkv, kh * a.k_head + 64 * c, row[p], f);
+          for (int c = a.key_chunks; c < qc; ++c) tp_load_2d(to + c * kPtKChunk, &mkr, 64 * (c - a.key_chunks), row[p], f);
+          for (int c = 0; c < vc; ++c) tp_load_2d(to + (qc + c) * kPtKChunk, &mkv, a.v_first + kh * a.vdim + 64 * c, row[p], f);
+        }
         issued = n + 1;
       }
       // no copy may be in flight when the CTA leaves
@@ -103,14 +116,16 @@ __global__ void __launch_bounds__(kPtThreads, 1)
     }
   } else if (warp == 5) {
     if (lane == 0) {
-      const uint32_t idesc_s = tp_idesc_bf16(kPtKeys), idesc_pv = tp_idesc_bf16(a.vdim) | (1u << 16);  // V: MN-major B operand
+      // V: MN-major B operand; columns past the value size hold whatever the copy brought and are not stored
+      const uint32_t idesc_s = tp_idesc_bf16(kPtKeys), idesc_pv = tp_idesc_bf16(64 * vc) | (1u << 16);
       auto issue_s = [&](int n) {
         const uint32_t k = sT + (uint32_t)(n % kPtStages) * stage_bytes;
         for (int c = 0; c < qc; ++c) {
           const uint64_t qd = tp_desc_k_sw128(sQ + c * kPtQChunk), kd = tp_desc_k_sw128(k + c * kPtKChunk);
 #pragma unroll
           for (int j = 0; j < 4; ++j)
-            tp_mma(tmem + kPtColS + 64 * (n & 1), qd + (uint64_t)(2 * j), kd + (uint64_t)(2 * j), idesc_s, (c | j) ? 1u : 0u);
+            if (64 * c + 16 * j < a.dim)
+              tp_mma(tmem + kPtColS + 64 * (n & 1), qd + (uint64_t)(2 * j), kd + (uint64_t)(2 * j), idesc_s, (c | j) ? 1u : 0u);
         }
         tp_commit(sfull + 8 * (n & 1));
       };
@@ -151,8 +166,25 @@ __global__ void __launch_bounds__(kPtThreads, 1)
     const int pos = first + q0 + tid;        // this thread's query
     const int warp_first = first + q0 + 32 * warp;
     float m_ref = 0.f, l = 0.f;
+    const float *bias = BIAS ? a.bias + (size_t)h * a.bias_len : nullptr;
     for (int n = 0; n < nt; ++n) {
       const int b = n & 1;
+      // entry i: distance near + i, lane l's key j at i = l + 63 - j
+      const int near = warp_first - n * kPtKeys - (kPtKeys - 1);
+      const bool flat = BIAS && near >= a.bias_len - 1;  // every distance is past the table's end
+      float flat_bias = 0.f;
+      if (BIAS) {
+        if (flat) {
+          flat_bias = bias[a.bias_len - 1] * kPtLog2e;
+        } else {
+#pragma unroll
+          for (int i = 0; i < 3; ++i) {
+            const int d = near + lane + 32 * i;
+            s_window[warp][lane + 32 * i] = d < 0 ? -INFINITY : bias[min(d, a.bias_len - 1)] * kPtLog2e;
+          }
+          __syncwarp();
+        }
+      }
       failed = !tp_wait(sfull + 8 * b, (uint32_t)((n >> 1) & 1));
       if (__any_sync(0xffffffffu, failed)) {
         failed = true;
@@ -165,7 +197,16 @@ __global__ void __launch_bounds__(kPtThreads, 1)
       tc_fence_before();
       __syncwarp();
       if (lane == 0) tp_arrive(sfree + 8 * b);
-      if (n * kPtKeys + kPtKeys - 1 > warp_first) {  // keys behind a query take no weight
+      if (BIAS) {
+        if (flat) {
+#pragma unroll
+          for (int j = 0; j < 64; ++j) r[j] = __float_as_uint(fmaf(__uint_as_float(r[j]), a.scale_log2, flat_bias));
+        } else {
+          const float *w = s_window[warp] + lane + 63;
+#pragma unroll
+          for (int j = 0; j < 64; ++j) r[j] = __float_as_uint(fmaf(__uint_as_float(r[j]), a.scale_log2, w[-j]));
+        }
+      } else if (n * kPtKeys + kPtKeys - 1 > warp_first) {  // keys behind a query take no weight
 #pragma unroll
         for (int j = 0; j < 64; ++j)
           if (n * kPtKeys + j > pos) r[j] = 0xff800000u;
@@ -178,7 +219,7 @@ __global__ void __launch_bounds__(kPtThreads, 1)
         x2 = fmaxf(x2, __uint_as_float(r[j + 2]));
         x3 = fmaxf(x3, __uint_as_float(r[j + 3]));
       }
-      const float mx = fmaxf(fmaxf(x0, x1), fmaxf(x2, x3)) * a.scale_log2;  // the scale is positive
+      const float mx = fmaxf(fmaxf(x0, x1), fmaxf(x2, x3)) * (BIAS ? 1.f : a.scale_log2);  // without a bias the scale is positive
       float alpha = 1.f;
       bool need = false;
       if (n == 0) {
@@ -192,7 +233,8 @@ __global__ void __launch_bounds__(kPtThreads, 1)
       float s0 = 0.f, s1 = 0.f;
 #pragma unroll
       for (int j = 0; j < 64; j += 2) {
-        const float p0 = pt_ex2(fmaf(__uint_as_float(r[j]), a.scale_log2, nm)), p1 = pt_ex2(fmaf(__uint_as_float(r[j + 1]), a.scale_log2, nm));
+        const float u = __uint_as_float(r[j]), v = __uint_as_float(r[j + 1]);
+        const float p0 = pt_ex2(BIAS ? u + nm : fmaf(u, a.scale_log2, nm)), p1 = pt_ex2(BIAS ? v + nm : fmaf(v, a.scale_log2, nm));
         s0 += p0;
         s1 += p1;
         r[j] = __float_as_uint(p0);
@@ -238,7 +280,8 @@ __global__ void __launch_bounds__(kPtThreads, 1)
     failed = __any_sync(0xffffffffu, failed);
     if (!failed) {
       tc_fence_after();
-      const float inv = 1.0f / l;
+      float inv = 1.0f / l;
+      if (a.gate && tid < nq) inv /= 1.0f + expf(-bf16_bits_to_f32(a.gate[(size_t)(q0 + tid) * a.ld_gate + h]));
       uint16_t *o = a.out + (size_t)(q0 + tid) * a.ldo + (size_t)h * a.vdim;
 #pragma unroll 1
       for (int c = 0; c < 2 * vc; ++c) {
@@ -248,6 +291,7 @@ __global__ void __launch_bounds__(kPtThreads, 1)
         if (tid < nq) {
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
+            if (32 * c + j >= a.vdim) break;
             uint32_t w[4];
 #pragma unroll
             for (int k = 0; k < 4; ++k) w[k] = pack_bf16x2(__uint_as_float(v[j + 2 * k]) * inv, __uint_as_float(v[j + 2 * k + 1]) * inv);
@@ -257,10 +301,28 @@ __global__ void __launch_bounds__(kPtThreads, 1)
       }
     }
   }
-  if (failed) atomicExch(&g_latent_prompt_error, 1u);
+  if (failed) atomicExch(&g_prompt_attn_error, 1u);
   tc_fence_before();
   __syncthreads();
   if (warp == 0) tp_tmem_free(tmem, kPtTmemCols);
+}
+
+bool prompt_attn_supports(int dim, int vdim) { return dim % 16 == 0 && dim <= 64 * kPtMaxQ && vdim % 16 == 0 && vdim <= 128; }
+
+int launch_prompt_attn(const CUtensorMap &mq, const CUtensorMap &mkv, const CUtensorMap &mkr, const PromptAttn &a, cudaStream_t stream) {
+  BLOK_REQUIRE(prompt_attn_supports(a.dim, a.vdim) && a.ldo % 8 == 0 && a.T >= 1 && a.n >= a.T && a.heads % a.share == 0, BLOK_ERR_SHAPE,
+               "prompt attention: heads of %d / %d, rows of %d outputs", a.dim, a.vdim, a.ldo);
+  const int qc = (a.dim + 63) / 64, vc = (a.vdim + 63) / 64;
+  const int smem = qc * kPtQChunk + kPtStages * (qc + vc) * kPtKChunk + 1024;
+  const dim3 grid((a.T + kPtRows - 1) / kPtRows, a.heads);
+  if (a.bias) {
+    BLOK_CUDA(cudaFuncSetAttribute(prompt_attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    prompt_attn_tc_kernel<true><<<grid, kPtThreads, smem, stream>>>(mq, mkv, mkr, a);
+  } else {
+    BLOK_CUDA(cudaFuncSetAttribute(prompt_attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    prompt_attn_tc_kernel<false><<<grid, kPtThreads, smem, stream>>>(mq, mkv, mkr, a);
+  }
+  return launch_status("prompt_attn_tc_kernel");
 }
 
 bool latent_prompt_tc_supports(const LatentShape &s) {
@@ -269,7 +331,6 @@ bool latent_prompt_tc_supports(const LatentShape &s) {
 
 int launch_latent_prompt_tc(const LatentShape &s, const uint16_t *q, const uint16_t *kv, const uint16_t *kr_all, int T, int n, uint16_t *o, int ldo,
                             cudaStream_t stream) {
-  BLOK_REQUIRE(ldo % 8 == 0, BLOK_ERR_SHAPE, "latent attention: rows of %d outputs", ldo);
   CUtensorMap mq, mkv, mkr;
   const int qw = s.heads * s.head(), kw = s.heads * (s.dim + s.vdim);
   int rc;
@@ -277,19 +338,57 @@ int launch_latent_prompt_tc(const LatentShape &s, const uint16_t *q, const uint1
   if ((rc = gemm_operand_map(q, T, qw, qw, kPtRows, &mq)) || (rc = gemm_operand_map(kv, n, kw, kw, kPtKeys, &mkv)) ||
       (rc = gemm_operand_map(kr_all, n, s.rot, s.rot, kPtKeys, &mkr)))
     return rc;
-  const PtArgs a = {o, T, n, ldo, s.heads, s.dim, s.rot, s.vdim, s.scale * 1.4426950408889634f};
-  const int qc = s.head() / 64, vc = s.vdim / 64;
-  const int smem = qc * kPtQChunk + kPtStages * (qc + vc) * kPtKChunk + 1024;
-  BLOK_CUDA(cudaFuncSetAttribute(latent_prompt_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  latent_prompt_tc_kernel<<<dim3((T + kPtRows - 1) / kPtRows, s.heads), kPtThreads, smem, stream>>>(mq, mkv, mkr, a);
-  return launch_status("latent_prompt_tc_kernel");
+  PromptAttn a;
+  a.out = o;
+  a.ldo = ldo;
+  a.T = T;
+  a.n = n;
+  a.heads = s.heads;
+  a.q_head = a.dim = s.head();
+  a.k_head = s.dim;
+  a.key_chunks = s.dim / 64;
+  a.v_first = s.heads * s.dim;
+  a.vdim = s.vdim;
+  a.scale_log2 = s.scale * kPtLog2e;
+  return launch_prompt_attn(mq, mkv, mkr, a, stream);
+}
+
+bool grouped_prompt_supports(const GroupedShape &s) { return (s.bias || s.scale > 0.f) && prompt_attn_supports(s.dim, s.vdim); }
+
+int launch_grouped_prompt(const GroupedShape &s, const GroupedQuery<uint16_t> &g, const void *pool, long pool_rows, const StackRows &r, int slot, int T,
+                          int n, cudaStream_t stream) {
+  BLOK_REQUIRE(g.ldq % 8 == 0 && r.page_rows % 32 == 0, BLOK_ERR_SHAPE, "prompt attention: rows of %d values, pages of %d", g.ldq, r.page_rows);
+  CUtensorMap mq, mkv;
+  const int box = r.page_rows % kPtKeys ? 32 : kPtKeys;  // a box stays inside a page
+  int rc;
+  if ((rc = gemm_operand_map(g.q, T, s.heads * s.dim, g.ldq, kPtRows, &mq)) || (rc = gemm_operand_map(pool, pool_rows, s.row(), s.row(), box, &mkv))) return rc;
+  PromptAttn a;
+  a.out = g.out;
+  a.ldo = g.ldo;
+  a.gate = g.gate;
+  a.ld_gate = g.ld_gate;
+  a.T = T;
+  a.n = n;
+  a.heads = s.heads;
+  a.share = s.heads / s.kv_heads;
+  a.q_head = a.k_head = a.dim = s.dim;
+  a.key_chunks = (s.dim + 63) / 64;
+  a.v_first = s.kv_heads * s.dim;
+  a.vdim = s.vdim;
+  a.scale_log2 = s.scale * kPtLog2e;
+  a.bias = s.bias;
+  a.bias_len = s.bias_len;
+  a.table = r.table + (size_t)slot * r.table_stride;
+  a.page_rows = r.page_rows;
+  a.box = box;
+  return launch_prompt_attn(mq, mkv, mkv, a, stream);
 }
 
 // *out becomes non-zero if a CTA has given up on a barrier since the last call (the flag is cleared).
-int latent_prompt_take_error(unsigned *out) {
+int prompt_attn_take_error(unsigned *out) {
   unsigned zero = 0;
-  BLOK_CUDA(cudaMemcpyFromSymbol(out, g_latent_prompt_error, sizeof(unsigned)));
-  if (*out) BLOK_CUDA(cudaMemcpyToSymbol(g_latent_prompt_error, &zero, sizeof(unsigned)));
+  BLOK_CUDA(cudaMemcpyFromSymbol(out, g_prompt_attn_error, sizeof(unsigned)));
+  if (*out) BLOK_CUDA(cudaMemcpyToSymbol(g_prompt_attn_error, &zero, sizeof(unsigned)));
   return BLOK_OK;
 }
 

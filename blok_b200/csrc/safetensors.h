@@ -74,7 +74,16 @@ class Safetensors {
     *out = &t;
     return BLOK_OK;
   }
+  const StoredTensor *find(const std::string &name) const {
+    auto it = tensors_.find(name);
+    return it == tensors_.end() ? nullptr : &it->second;
+  }
   int read(const StoredTensor &t, void *dst) const { return read_at(t.at, dst, t.bytes); }
+  // `bytes` of the tensor from byte `from` on; the caller has checked its shape
+  int read(const StoredTensor &t, void *dst, uint64_t from, uint64_t bytes) const {
+    BLOK_REQUIRE(from <= t.bytes && bytes <= t.bytes - from, BLOK_ERR_SHAPE, "%s: a part outside its tensor", path_.c_str());
+    return read_at(t.at + from, dst, bytes);
+  }
 
  private:
   int fd_ = -1;

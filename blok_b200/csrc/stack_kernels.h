@@ -48,16 +48,51 @@ struct StreamsStep {
 };
 int launch_streams_step(const StreamsStep &a, cudaStream_t stream);
 
-// ---- linear attention with a fixed decay per head (linear_attn.cu) ----
+// ---- one residual between sandwiched sublayers (residual_norm.cu) ----
+constexpr int kMaxNormWidth = 32768;
+struct ResidualNorm {
+  int T = 0, width = 0, true_width = 0;  // width: padded, zero in the padding
+  float *x = nullptr;                    // [T, width]
+  // x from the embeddings when ids is set: embed_scale * embed[id] + the pair's row + the position's sinusoid
+  const uint32_t *ids = nullptr;
+  const uint16_t *embed = nullptr, *bigram = nullptr;  // bf16 [vocab, width], [buckets + 1, width] or NULL
+  int vocab = 0, buckets = 0;
+  long mul_prev = 0, mul_cur = 0;
+  float embed_scale = 1.f;
+  const double *turns = nullptr;         // [width / 2] turns per position of every pair of columns, or NULL
+  const int *pos = nullptr, *slot_of = nullptr;
+  bool chunk = false;                    // rows are consecutive tokens of one sequence
+  uint32_t *last_ids = nullptr;          // [slots] the newest token of every sequence
+  const uint32_t *keep_ids = nullptr;    // set: last_ids takes in this call's newest tokens (in a later launch than ids)
+  // else x += mult * layer_norm(y) * post_w (post_w NULL: += mult * y) when y is set
+  const float *y = nullptr;              // [T, width]
+  const float *post_w = nullptr;
+  float mult = 1.f, eps = 0.f;
+  float *copy = nullptr;                 // [T, true_width]: x (for parity checks)
+  // h = layer_norm(x) * norm_w, Act [T, width]
+  const float *norm_w = nullptr;
+  void *h = nullptr;
+  bool h_f32 = false;
+};
+int launch_residual_norm(const ResidualNorm &a, cudaStream_t stream);
+
+// ---- linear attention with a decay per head, fixed or per token (linear_attn.cu) ----
 enum { GATE_SILU = 0, GATE_SIGMOID = 1 };
 struct LinearAttn {
   int heads = 0, dim = 0, vdim = 0;  // padded: multiples of 16
   const void *qkvg = nullptr;        // Act [T, ld]: q | k | v | g, head by head
+  int share = 1;                     // so many heads share one head of q and k
+  bool v_first = false;              // Act [T, ld]: v | k | q
   int ld = 0;
   bool f32 = false;
   bool silu_qkv = false;             // q, k and v go through SiLU (rounded to Act) when they are read
   float k_scale = 1.f;
   const float *decay_pow = nullptr;  // [heads, kLinChunk + 1]: decay^i
+  // decays per token instead: [heads, token_ld] of (key scale, log decay, the log decays' running sum inside the token's chunk
+  // of kLinChunk in two parts), and o += skip[head] v
+  const float4 *token = nullptr;
+  int token_ld = 0;
+  const float *skip = nullptr;       // [heads]
   float *state = nullptr;            // fp32 [slots, heads, dim, vdim]
   float *o = nullptr;                // fp32 [T, heads * vdim]
   float *chunk_state = nullptr;      // scratch [chunks, heads, dim, vdim] of the chunked form
@@ -83,6 +118,24 @@ struct GatedNorm {
   bool f32 = false;
 };
 int launch_gated_norm(const GatedNorm &a, int T, cudaStream_t stream);
+// out = rmsnorm(o * silu(g)) * w over `parts` equal parts of the heads * true_vdim true columns (per_head, gate: unused).
+int launch_gate_then_norm(const GatedNorm &a, int parts, int T, cudaStream_t stream);
+
+// ---- inputs of a selective state space (state_space.cu) ----
+struct StateInputs {
+  int heads = 0, channels = 0, taps = 0;  // channels: padded, a multiple of 16
+  const void *proj = nullptr;             // Act [T, ld]: anything | channels at `first` | anything | steps at dt_at
+  int ld = 0, first = 0, dt_at = 0;
+  bool f32 = false;
+  const float *conv_w = nullptr, *conv_b = nullptr;   // [taps, channels] (current token last), [channels]
+  const float *dt_bias = nullptr, *rate = nullptr;    // [heads]; rate = -exp(log rate)
+  void *ring = nullptr;                   // Act [slots, taps, channels]: the input at position p lies at p % taps
+  void *out = nullptr;                    // Act [T, channels]: silu(conv + b)
+  float4 *token = nullptr;                // [heads, token_ld], see LinearAttn
+  int token_ld = 0;
+};
+// Rows are the next token of T sequences, or (chunk) T consecutive tokens of one.
+int launch_state_inputs(const StateInputs &a, const StackRows &r, int T, bool chunk, cudaStream_t stream);
 
 // ---- latent attention over a paged cache of rows [latent | rotated key] (latent_attn.cu) ----
 struct LatentShape {
@@ -117,6 +170,39 @@ bool latent_prompt_supports(const LatentShape &s);
 int launch_latent_prompt(const LatentShape &s, const uint16_t *q, const uint16_t *kv, const uint16_t *kr_all, int T, int n, uint16_t *o, int ldo,
                          cudaStream_t stream);
 
+// ---- grouped softmax attention over a paged cache of rows [keys | values] (grouped_attn.cu, prompt_attn_tc.cu) ----
+struct GroupedShape {
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0;  // padded: dim a multiple of 32, vdim of 16
+  int true_dim = 0;
+  float scale = 1.f, eps = 0.f;
+  const float *bias = nullptr;  // [heads, bias_len] by distance, the last entry for every distance from there on; or NULL
+  int bias_len = 0;
+  __host__ __device__ int row() const { return kv_heads * (dim + vdim); }  // a cached row
+};
+template <typename Act>
+struct GroupedQuery {
+  const Act *q = nullptr;     // [T, ldq]: head by head
+  int ldq = 0;
+  const Act *gate = nullptr;  // [T, ld_gate], one value per head, before the sigmoid; or NULL
+  int ld_gate = 0;
+  Act *out = nullptr;         // [T, ldo]: head by head
+  int ldo = 0;
+};
+// qkv Act [T, ld]: q | k | v.  q is normed in place over all heads (q_norm NULL: left alone), k likewise, and the row appended to
+// the pool (Act [pages, page_rows, row]; NULL: q only).
+int launch_grouped_append(const GroupedShape &s, void *qkv, int ld, const float *q_norm, const float *k_norm, const StackRows &r, int T, void *pool,
+                          bool f32, cudaStream_t stream);
+// Entry i attends to positions 0..pos[i].  part_o fp32 [max_parts, heads, vdim], part_ml fp32 [max_parts, heads, 2], finite at the
+// first call (see launch_latent_attend).
+size_t grouped_attend_max_parts(const GroupedShape &s, int T, long max_ctx);
+int launch_grouped_attend(const GroupedShape &s, const GroupedQuery<uint16_t> &a, const void *pool, const StackRows &r, int T, long max_ctx,
+                          float *part_o, float *part_ml, cudaStream_t stream);
+int launch_grouped_attend_f32(const GroupedShape &s, const GroupedQuery<float> &a, const void *pool, const StackRows &r, int T, cudaStream_t stream);
+// T tokens of the sequence in `slot` at positions n - T .. n - 1; every row of the pool must hold finite values.
+bool grouped_prompt_supports(const GroupedShape &s);
+int launch_grouped_prompt(const GroupedShape &s, const GroupedQuery<uint16_t> &a, const void *pool, long pool_rows, const StackRows &r, int slot, int T,
+                          int n, cudaStream_t stream);
+
 // ---- experts chosen by a table of token ids (table_experts.cu) ----
 struct ExpertPlan {          // of one layer and call
   int *at = nullptr;         // [T * top] row of assignment (t, k) in expert order
@@ -145,5 +231,7 @@ struct GemmF32 {
   long w_stride = 0, x_stride = 0, y_stride = 0;  // between batches
 };
 int launch_gemm_f32(const GemmF32 &g, cudaStream_t stream);
+// out[t, r] = silu(x[t, r]) * x[t, cols + r], x fp32 [T, 2 cols]
+int launch_swiglu_f32(const float *x, float *out, int cols, int T, cudaStream_t stream);
 
 }  // namespace blok

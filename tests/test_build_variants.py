@@ -50,7 +50,7 @@ def test_fused_kernel_registers_and_spills(tmp_path):
     # 288 threads, two CTAs per SM (tensor memory and shared memory are sized for two): 113 registers at most
     ("wgemm_tc.cu", "wgemm_tc_kernel", 112, 16),
     # 192 threads: the softmax rows of the prompt kernel live in registers; two GEMM CTAs per SM at the 128-row tile
-    ("latent_prompt_tc.cu", "latent_prompt_tc_kernel", 255, 0),
+    ("prompt_attn_tc.cu", "prompt_attn_tc_kernel", 255, 0),
     ("gemm_tma.cu", "gemm_tma_kernel", 80, 0),
     # 256 threads, two CTAs per SM
     ("linear_attn.cu", "linear_chunk_out_kernel", 128, 0),
