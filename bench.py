@@ -351,28 +351,102 @@ def nomozen_bytes(c, batch, ctx):
     return total + c["vocab"] * W * 2
 
 
+PAMOPEL_SIZES = {
+    # width, state-space heads (of 64, twice the width together), attention heads and key heads (of 128), feed-forward size
+    "small": dict(width=2048, heads=64, q_heads=16, kv_heads=4, ff=8192),
+    "large": dict(width=4096, heads=128, q_heads=32, kv_heads=8, ff=14336),
+}
+
+
+def pamopel_config(width, heads, q_heads, kv_heads, ff, vocab=32768):
+    """A four-layer Pamopel model of a real model's layer sizes: state space, attention, attention that borrows keys, state space."""
+    mlp = {"kind": "dense", "ff": ff}
+    state = {"heads": heads, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    attn = {"heads": q_heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "bias_max": 128}
+    return {"architecture": "Pamopel", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "logit_scale": 1.0,
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+            "layers": [{"type": "mamba2", "mixer": state, "mlp": mlp}, {"type": "attention", "mixer": attn, "mlp": mlp},
+                       {"type": "attention", "mixer": dict(attn, kv_from=1), "mlp": mlp}, {"type": "mamba2", "mixer": state, "mlp": mlp}]}
+
+
+def pamopel_like_nomozen(width, heads, q_heads, kv_heads, ff, vocab=32768):
+    """The Nomozen model of the same layers: retention with states of the same shape, latent attention with as many heads of the
+    same size, one expert that every token takes, one residual stream."""
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": 1, "top": 1}}
+    linear = {"heads": heads, "dim": 128, "vdim": 64, "decay": [1 - 2.0 ** -(5 + 5 * h / heads) for h in range(heads)]}
+    latent = {"heads": q_heads, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 1536, "scale": 128 ** -0.5,
+              "rot": {"base": 50000.0, "dims": 64}}
+    return {"architecture": "Nomozen", "width": width, "vocab": vocab, "streams": 1, "norm": {"eps": 1e-5},
+            "layers": [dict(l, mlp=mlp) for l in ({"type": "retention", "mixer": linear}, {"type": "latent_attention", "mixer": latent},
+                                                  {"type": "latent_attention", "mixer": latent}, {"type": "lightning", "mixer": linear})]}
+
+
+def pamopel_bytes(c, batch, ctx):
+    """Algorithmic bytes of one decode step: every weight once, states, cached rows and convolution inputs once."""
+    W, total = c["width"], 0
+    for l in c["layers"]:
+        m = l["mixer"]
+        if l["type"] == "attention":
+            q, kv = m["heads"] * m["dim"], m["kv_heads"] * (m["dim"] + m["vdim"])
+            total += 2 * W * (q + (0 if "kv_from" in m else kv) + m["heads"] + m["heads"] * m["vdim"]) + batch * ctx * kv * 2
+        else:
+            inner, bc = m["heads"] * m["vdim"], 2 * m["groups"] * m["state"]
+            total += 2 * W * (2 * inner + bc + m["heads"] + inner) + batch * (inner * m["state"] * 8 + (inner + bc) * m["conv"] * 2)
+        total += 2 * 3 * W * l["mlp"]["ff"] + 4 * batch * W * 4
+    return total + c["vocab"] * W * 2
+
+
+def pamopel_prompt_flops(c, T):
+    """Multiply-adds of a T-token prompt's products and attention, each counted once, times two."""
+    W, total = c["width"], 0
+    for l in c["layers"]:
+        m = l["mixer"]
+        if l["type"] == "attention":
+            q, kv = m["heads"] * m["dim"], m["kv_heads"] * (m["dim"] + m["vdim"])
+            total += T * W * (q + (0 if "kv_from" in m else kv) + m["heads"] * m["vdim"]) + T * T // 2 * m["heads"] * (m["dim"] + m["vdim"])
+        else:
+            inner, bc = m["heads"] * m["vdim"], 2 * m["groups"] * m["state"]
+            total += T * W * (3 * inner + bc) + 2 * T * inner * m["state"]
+        total += T * 3 * W * l["mlp"]["ff"]
+    return 2 * total
+
+
 def nomozen_workload(a, device, steps, warmup):
-    """Decode and prompt throughput of a Nomozen model beside the library's Kimi model at equal sizes (four layers each, the
-    same width, attention, expert count and size; Kimi's experts are INT4 and have three matrices), one GPU.  --impl-only
-    runs one of the two (profiler launch lists)."""
-    import torch
+    """A Nomozen model beside the library's Kimi model (Kimi's experts are INT4 and have three matrices)."""
     from blok_b200 import lib
     size = NOMOZEN_SIZES[a.size]
-    B, ctx, P = a.batch, a.ctx, a.prompt
     cfg = nomozen_config(**size)
-    vocab = cfg["vocab"]
+    kimi = lambda vocab, **o: lib.Model(seed=4, layers=4, first_dense=0, hidden=size["width"], vocab=vocab, inter=size["ff"], experts=size["experts"],
+                                        topk=size["top"], shared_inter=size["ff"], kv_page_rows=64, **dict(o, prefill_chunk=64))
+    return model_workload(a, device, steps, warmup, "Nomozen", size, cfg["vocab"], {"nomozen": cfg, "kimi": kimi}, nomozen_bytes)
+
+
+def pamopel_workload(a, device, steps, warmup):
+    """A Pamopel model beside the library's Nomozen model."""
+    size = PAMOPEL_SIZES[a.size]
+    cfg = pamopel_config(**size)
+    return model_workload(a, device, steps, warmup, "Pamopel", size, cfg["vocab"], {"pamopel": cfg, "nomozen": pamopel_like_nomozen(**size)}, pamopel_bytes,
+                          pamopel_prompt_flops)
+
+
+def model_workload(a, device, steps, warmup, title, size, vocab, models, step_bytes, prompt_flops=None):
+    """Decode and prompt throughput of the first of two models beside the second at equal sizes (four layers each, the same width,
+    heads, feed-forward and vocabulary), one GPU.  models: name -> config.json (a dict), or a function that makes the model.
+    --impl-only runs one of the two (profiler launch lists)."""
+    import torch
+    from blok_b200 import lib
+    B, ctx, P = a.batch, a.ctx, a.prompt
     max_ctx = max(ctx, P) + steps + max(warmup, 3) + 16
     pages = B * ((max_ctx + 63) // 64) + ((P + 63) // 64)
     peak, peak_kind = measured_peak()
-    kinds = {"nomozen": lambda: lib.Model.open_synthetic(cfg, seed=4, max_batch=B + 1, max_ctx=max_ctx, prefill_chunk=min(2048, max(P, ctx)), kv_pages=pages),
-             "kimi": lambda: lib.Model(seed=4, layers=4, first_dense=0, hidden=size["width"], vocab=vocab, inter=size["ff"], experts=size["experts"],
-                                       topk=size["top"], shared_inter=size["ff"], max_batch=B + 1, max_ctx=max_ctx, prefill_chunk=64,
-                                       kv_page_rows=64, kv_pages=pages)}
+    options = dict(max_batch=B + 1, max_ctx=max_ctx, prefill_chunk=min(2048, max(P, ctx)), kv_pages=pages)
+    first = next(iter(models))
     sampler = ClockSampler(device.index or 0)
     sampler.start()
     out, launches = {}, 0
-    for kind in ([a.impl_only] if a.impl_only else ["nomozen", "kimi"]):
-        model = kinds[kind]()
+    for kind in ([a.impl_only] if a.impl_only else models):
+        made = models[kind]
+        model = lib.Model.open_synthetic(made, seed=4, **options) if isinstance(made, dict) else made(vocab, **options)
         side = torch.cuda.Stream()
         torch.cuda.synchronize()
         with torch.cuda.stream(side):
@@ -396,6 +470,8 @@ def nomozen_workload(a, device, steps, warmup):
                 launches += lib.kernel_launch_count() - l0
                 rec["prefill_ms"] = e0.elapsed_time(e1) / n
                 rec["prefill_tok_per_s"] = P / (rec["prefill_ms"] * 1e-3)
+                if kind == first and prompt_flops:
+                    rec["prefill_tflops"] = prompt_flops(made, P) / (rec["prefill_ms"] * 1e-3) / 1e12
             if ctx:
                 for b in range(B):
                     model.prefill_slot(b, prompts[b % 4][:ctx])
@@ -413,21 +489,21 @@ def nomozen_workload(a, device, steps, warmup):
                 launches += lib.kernel_launch_count() - l0
                 rec["decode_ms"] = e0.elapsed_time(e1) / steps
                 rec["decode_tok_per_s"] = B / (rec["decode_ms"] * 1e-3)
-                if kind == "nomozen":
-                    alg = nomozen_bytes(cfg, B, ctx)
+                if kind == first:
+                    alg = step_bytes(made, B, ctx)
                     rec["decode_roofline"] = {"bound": "hbm", "bytes": alg, "achieved": alg / (rec["decode_ms"] * 1e-3) / 1e9, "peak": peak,
                                               "unit": "GB/s", "frac": alg / (rec["decode_ms"] * 1e-3) / 1e9 / peak, "peak_kind": peak_kind}
             model.check()
         model.close()
         out[kind] = rec
     clocks = sampler.stop()
-    main = out.get("nomozen", out.get("kimi"))
+    main = out.get(first) or next(iter(out.values()))
     print(json.dumps({
-        "metric": "decode tok/s, 4-layer Nomozen model (batch %d, ctx %d)" % (B, ctx), "value": main.get("decode_tok_per_s"), "unit": "tok/s",
+        "metric": "decode tok/s, 4-layer %s model (batch %d, ctx %d)" % (title, B, ctx), "value": main.get("decode_tok_per_s"), "unit": "tok/s",
         "n_gpus": 1, "steps": steps, "warmup": warmup, "ms_per_step": main.get("decode_ms"), "higher_is_better": True, "scaling": "weak",
         "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-        "config": {"workload": "Nomozen beside Kimi's model at equal size (%s: %s), four layers each, %d-token prompts, paged caches" %
-                               (a.size, json.dumps(size), P),
+        "config": {"workload": "%s at equal size (%s: %s), four layers each, %d-token prompts, paged caches" %
+                               (" beside ".join(models), a.size, json.dumps(size), P),
                    "l2": "a step reads more weights than the L2 holds; prompts rotated"},
         **out, "gpu_launches": int(launches), "clocks": clocks}))
     return 0
@@ -706,14 +782,14 @@ def main():
     ap.add_argument("--experts", type=int, default=384,
                     help="routed experts per layer; below 384 the run is a reduced case for profiler captures, "
                          "not the benchmark configuration, and the line says so")
-    ap.add_argument("--size", default="large", choices=sorted(NOMOZEN_SIZES), help="layer sizes of the `nomozen` workload")
-    ap.add_argument("--ctx", type=int, default=4096, help="cached tokens per sequence of the `nomozen` workload (0: no decoding)")
-    ap.add_argument("--prompt", type=int, default=1024, help="prompt length of the `nomozen` workload (0: no prompts)")
-    ap.add_argument("--impl-only", default=None, choices=["nomozen", "kimi"], help="one side of the `nomozen` workload")
-    ap.add_argument("--workload", default="decode", choices=["decode", "expert", "batched64", "batched2048", "mla4096", "mla32768", "model", "model61", "prefill512", "gemv", "nomozen"],
+    ap.add_argument("--size", default="large", choices=sorted(NOMOZEN_SIZES), help="layer sizes of the `nomozen` and `pamopel` workloads")
+    ap.add_argument("--ctx", type=int, default=4096, help="cached tokens per sequence of the `nomozen` and `pamopel` workloads (0: no decoding)")
+    ap.add_argument("--prompt", type=int, default=1024, help="prompt length of the `nomozen` and `pamopel` workloads (0: no prompts)")
+    ap.add_argument("--impl-only", default=None, choices=["nomozen", "kimi", "pamopel"], help="one side of the `nomozen` or `pamopel` workload")
+    ap.add_argument("--workload", default="decode", choices=["decode", "expert", "batched64", "batched2048", "mla4096", "mla32768", "model", "model61", "prefill512", "gemv", "nomozen", "pamopel"],
                     help="decode = config 1 (the default, the headline metric); batched* = config 2 (expert parallel "
                          "when --gpus > 1); mla* = config 3 (attention block, batch 8); nomozen = a Nomozen model beside "
-                         "Kimi's at equal size, one GPU (--size, --batch, --ctx, --prompt)")
+                         "Kimi's at equal size, pamopel = a Pamopel model beside Nomozen's, one GPU (--size, --batch, --ctx, --prompt)")
     a = ap.parse_args()
 
     import torch
@@ -750,8 +826,9 @@ def main():
     if world > 1:
         dist.init_process_group("nccl", device_id=device)
     lib.load()
-    if a.workload == "nomozen":
-        return nomozen_workload(a, device, steps if a.steps is not None else 20, warmup if a.warmup is not None else 5)
+    if a.workload in ("nomozen", "pamopel"):
+        run = nomozen_workload if a.workload == "nomozen" else pamopel_workload
+        return run(a, device, steps if a.steps is not None else 20, warmup if a.warmup is not None else 5)
     if a.workload != "decode":
         return other_workload(a, rank, world, device, steps if a.steps is not None else 20, warmup if a.warmup is not None else 5)
 

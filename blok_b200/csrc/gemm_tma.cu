@@ -154,22 +154,23 @@ __global__ void __launch_bounds__(kGtThreads)
             }
           }
         }
-      } else
+      } else {
 #pragma unroll 1
-      for (int c0 = 0; c0 < BN; c0 += 32) {
-        if (n0 + c0 >= a.R) break;
-        uint32_t v[32];
-        tmem_ld32(tmem + ((uint32_t)(32 * warp) << 16) + c0, v);
-        tmem_wait_ld();
-        if (r < count) {
+        for (int c0 = 0; c0 < BN; c0 += 32) {
+          if (n0 + c0 >= a.R) break;
+          uint32_t v[32];
+          tmem_ld32(tmem + ((uint32_t)(32 * warp) << 16) + c0, v);
+          tmem_wait_ld();
+          if (r < count) {
 #pragma unroll
-          for (int j = 0; j < 32; j += 4) {
-            const int col = n0 + c0 + j;
-            if (col < a.R) {  // R is a multiple of 4
-              float f0 = __uint_as_float(v[j]), f1 = __uint_as_float(v[j + 1]), f2 = __uint_as_float(v[j + 2]), f3 = __uint_as_float(v[j + 3]);
-              if (ACT != GEMM_ACT_SILU || col < a.act_cols) f0 = gt_act<ACT>(f0), f1 = gt_act<ACT>(f1), f2 = gt_act<ACT>(f2), f3 = gt_act<ACT>(f3);
-              if (F32) *reinterpret_cast<float4 *>(static_cast<float *>(a.out) + o + col) = make_float4(f0, f1, f2, f3);
-              else *reinterpret_cast<uint2 *>(static_cast<uint16_t *>(a.out) + o + col) = make_uint2(pack_bf16x2(f0, f1), pack_bf16x2(f2, f3));
+            for (int j = 0; j < 32; j += 4) {
+              const int col = n0 + c0 + j;
+              if (col < a.R) {  // R is a multiple of 4
+                float f0 = __uint_as_float(v[j]), f1 = __uint_as_float(v[j + 1]), f2 = __uint_as_float(v[j + 2]), f3 = __uint_as_float(v[j + 3]);
+                if (ACT != GEMM_ACT_SILU || col < a.act_cols) f0 = gt_act<ACT>(f0), f1 = gt_act<ACT>(f1), f2 = gt_act<ACT>(f2), f3 = gt_act<ACT>(f3);
+                if (F32) *reinterpret_cast<float4 *>(static_cast<float *>(a.out) + o + col) = make_float4(f0, f1, f2, f3);
+                else *reinterpret_cast<uint2 *>(static_cast<uint16_t *>(a.out) + o + col) = make_uint2(pack_bf16x2(f0, f1), pack_bf16x2(f2, f3));
+              }
             }
           }
         }

@@ -731,6 +731,107 @@ def latent_prompt(q, kv, k_rot, dim, vdim, scale):
     return o
 
 
+def residual_norm(x, y, post_w, mult, norm_w, eps, true_width, f32=True):
+    """blok_residual_norm: x fp32 [T, width], updated in place; returns h."""
+    T, width = x.shape
+    h = torch.empty((T, width), dtype=torch.float32 if f32 else torch.bfloat16, device=x.device)
+    _check(load().blok_residual_norm(_ptr(x, torch.float32, "x"), _ptr(y), _ptr(post_w), C.c_float(mult), _ptr(norm_w), C.c_float(eps), C.c_int(T),
+                                     C.c_int(width), C.c_int(true_width), _ptr(h), C.c_int(bool(f32)), _stream()))
+    return h
+
+
+def token_embedding(ids, last_ids, slot_of, pos, chunk, keep, embed, bigram, buckets, mul_prev, mul_cur, scale, turns, true_width):
+    """blok_token_embedding: ids int32 [T], tables bf16 -> x fp32 [T, width]; last_ids int32 [slots] is updated with keep."""
+    T, width = ids.numel(), embed.shape[1]
+    x = torch.empty((T, width), dtype=torch.float32, device=ids.device)
+    _check(load().blok_token_embedding(_ptr(ids, torch.int32, "ids"), _ptr(last_ids), _ptr(slot_of, torch.int32, "slot_of"), _ptr(pos, torch.int32, "pos"),
+                                       C.c_int(bool(chunk)), C.c_int(bool(keep)), _ptr(embed, torch.bfloat16, "embed"), C.c_int(embed.shape[0]),
+                                       _ptr(bigram), C.c_int(buckets), C.c_long(mul_prev), C.c_long(mul_cur), C.c_float(scale), _ptr(turns), C.c_int(T),
+                                       C.c_int(width), C.c_int(true_width), _ptr(x), _stream()))
+    return x
+
+
+def state_inputs(proj, first, dt_at, heads, conv_w, conv_b, dt_bias, rate, ring, slot_of, pos, chunk):
+    """blok_state_inputs: proj [T, ld], conv_w fp32 [taps, channels], ring [slots, taps, channels] updated ->
+    (out [T, channels], token fp32 [heads, T, 4])."""
+    T, ld = proj.shape
+    taps, channels = conv_w.shape
+    out = torch.empty((T, channels), dtype=proj.dtype, device=proj.device)
+    token = torch.empty((heads, T, 4), dtype=torch.float32, device=proj.device)
+    _check(load().blok_state_inputs(_ptr(proj), C.c_int(proj.dtype == torch.float32), C.c_int(ld), C.c_int(first), C.c_int(dt_at), C.c_int(heads),
+                                    C.c_int(channels), C.c_int(taps), _ptr(conv_w), _ptr(conv_b), _ptr(dt_bias), _ptr(rate), _ptr(ring),
+                                    _ptr(slot_of, torch.int32, "slot_of"), _ptr(pos, torch.int32, "pos"), C.c_int(T), C.c_int(bool(chunk)), _ptr(out),
+                                    _ptr(token), C.c_int(T), _stream()))
+    return out, token
+
+
+def selective_state(xbc, heads, groups, state_dim, vdim, token, skip, state, slot=0, first_pos=0, slot_of=None, pos=None):
+    """blok_selective_state: xbc [T, ld], token fp32 [heads, T, 4], state fp32 [slots, heads, state_dim, vdim] updated -> o fp32."""
+    T, ld = xbc.shape
+    f = load().blok_linear_attention_scratch_bytes
+    f.restype = C.c_size_t
+    scratch = torch.empty(f(heads, state_dim, vdim, T), dtype=torch.uint8, device=xbc.device)
+    o = torch.empty((T, heads * vdim), dtype=torch.float32, device=xbc.device)
+    _check(load().blok_selective_state(_ptr(xbc), C.c_int(xbc.dtype == torch.float32), C.c_int(ld), C.c_int(heads), C.c_int(groups), C.c_int(state_dim),
+                                       C.c_int(vdim), _ptr(token, torch.float32, "token"), C.c_int(token.shape[1]), _ptr(skip), _ptr(state, torch.float32, "state"),
+                                       C.c_int(slot), C.c_int(first_pos), C.c_int(T), _ptr(slot_of), _ptr(pos), _ptr(o), _ptr(scratch), _stream()))
+    return o
+
+
+def gate_then_norm(o, gate, heads, vdim, true_vdim, parts, eps, w=None):
+    """blok_gate_then_norm: o fp32 [T, heads * vdim], gate bf16 or fp32 of the same shape."""
+    out = torch.empty_like(gate)
+    _check(load().blok_gate_then_norm(_ptr(o, torch.float32, "o"), _ptr(gate), C.c_int(gate.shape[1]), _ptr(w), C.c_int(heads), C.c_int(vdim),
+                                      C.c_int(true_vdim), C.c_int(parts), C.c_float(eps), C.c_int(o.shape[0]), _ptr(out), C.c_int(out.shape[1]),
+                                      C.c_int(gate.dtype == torch.float32), _stream()))
+    return out
+
+
+def grouped_append(qkv, heads, kv_heads, dim, true_dim, vdim, q_norm, k_norm, eps, table, slot_of, pos, pool):
+    """blok_grouped_append: qkv [T, ld] (q normed in place), pool [pages, page_rows, row] or None."""
+    _check(load().blok_grouped_append(_ptr(qkv), C.c_int(qkv.dtype == torch.float32), C.c_int(qkv.shape[1]), C.c_int(heads), C.c_int(kv_heads),
+                                      C.c_int(dim), C.c_int(true_dim), C.c_int(vdim), _ptr(q_norm), _ptr(k_norm), C.c_float(eps), _ptr(table),
+                                      C.c_int(table.shape[1]), C.c_int(pool.shape[1] if pool is not None else 0), _ptr(slot_of), _ptr(pos),
+                                      C.c_int(qkv.shape[0]), _ptr(pool), _stream()))
+
+
+def grouped_attend(q, pool, table, slot_of, pos, kv_heads, vdim, scale, max_ctx, bias=None, gate=None):
+    """blok_grouped_attend: q [T, heads, dim], pool [pages, page_rows, row], bias fp32 [heads, n], gate [T, heads] ->
+    [T, heads, vdim]."""
+    T, heads, dim = q.shape
+    f = load().blok_grouped_attend_workspace_bytes
+    f.restype = C.c_size_t
+    ws = torch.zeros(max(16, f(heads, kv_heads, dim, vdim, T, C.c_long(max_ctx))), dtype=torch.uint8, device=q.device)
+    out = torch.empty((T, heads, vdim), dtype=q.dtype, device=q.device)
+    _check(load().blok_grouped_attend(_ptr(q), C.c_int(q.dtype == torch.float32), C.c_int(heads * dim), _ptr(gate), C.c_int(heads), _ptr(pool),
+                                      _ptr(table, torch.int32, "table"), C.c_int(table.shape[1]), C.c_int(pool.shape[1]),
+                                      _ptr(slot_of, torch.int32, "slot_of"), _ptr(pos, torch.int32, "pos"), C.c_int(heads), C.c_int(kv_heads), C.c_int(dim),
+                                      C.c_int(vdim), C.c_float(scale), _ptr(bias), C.c_int(0 if bias is None else bias.shape[1]), C.c_int(T),
+                                      C.c_long(max_ctx), _ptr(out), C.c_int(heads * vdim), _ptr(ws), _stream()))
+    return out
+
+
+def grouped_prompt(q, pool, table, slot, n, kv_heads, vdim, scale, bias=None, gate=None):
+    """blok_grouped_prompt: q bf16 [T, heads, dim] at positions n - T .. n - 1 of the sequence in `slot` -> [T, heads, vdim]."""
+    T, heads, dim = q.shape
+    out = torch.empty((T, heads, vdim), dtype=torch.bfloat16, device=q.device)
+    _check(load().blok_grouped_prompt(_ptr(q, torch.bfloat16, "q"), C.c_int(heads * dim), _ptr(gate), C.c_int(heads), _ptr(pool, torch.bfloat16, "pool"),
+                                      C.c_long(pool.shape[0] * pool.shape[1]), _ptr(table, torch.int32, "table"), C.c_int(table.shape[1]),
+                                      C.c_int(pool.shape[1]), C.c_int(slot), C.c_int(heads), C.c_int(kv_heads), C.c_int(dim), C.c_int(vdim),
+                                      C.c_float(scale), _ptr(bias), C.c_int(0 if bias is None else bias.shape[1]), C.c_int(T), C.c_int(n), _ptr(out),
+                                      C.c_int(heads * vdim), _stream()))
+    return out
+
+
+def gemm_swiglu(x, w):
+    """blok_gemm_swiglu: x bf16 [T, K], w bf16 [2 R, K] (gate rows, then up rows) -> bf16 [T, R]."""
+    R = w.shape[0] // 2
+    out = torch.empty((x.shape[0], R), dtype=torch.bfloat16, device=x.device)
+    _check(load().blok_gemm_swiglu(_ptr(x, torch.bfloat16, "x"), _ptr(w, torch.bfloat16, "w"), C.c_int(x.shape[0]), C.c_int(R), C.c_int(x.shape[1]),
+                                   _ptr(out), _stream()))
+    return out
+
+
 def gemm_bf16(x, w, relu2=False, f32=True):
     """blok_gemm_bf16: x [T, K], w [R, K] bf16 -> [T, R] fp32 (or bf16)."""
     out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32 if f32 else torch.bfloat16, device=x.device)

@@ -531,6 +531,67 @@ int blok_latent_attend(const void *q, const void *pool, const int *table, int ta
  * kv [n, heads * dim | heads * vdim], k_rot [n, rot], o [T, ld_out].  dim + rot and vdim at most 256. */
 int blok_latent_prompt(const blok_bf16_t *q, const blok_bf16_t *kv, const blok_bf16_t *k_rot, int heads, int dim, int rot,
                        int vdim, float scale, int T, int n, blok_bf16_t *o, int ld_out, blok_stream_t stream);
+/* One residual between sandwiched sublayers: x += mult * layer_norm(y) * post_w, then h = layer_norm(x) * norm_w (layer norms
+ * without a bias, over true_width of the rows' width values, zeros behind them).  y NULL: x stays; post_w NULL: y is added
+ * without a norm.  x and y fp32 [T, width], h bf16 or fp32.  width is a multiple of 4, at most 32768. */
+int blok_residual_norm(float *x, const float *y, const float *post_w, float mult, const float *norm_w, float eps, int T,
+                       int width, int true_width, void *h, int f32, blok_stream_t stream);
+/* x[t] = scale * embed[ids[t]] + bigram[(previous * mul_prev + ids[t] * mul_cur) mod buckets] (row `buckets` at position 0) +
+ * the sinusoid of the position (entry 2i sin, 2i + 1 cos of pos[t] * 2 pi * turns[i]).  bigram and turns may be NULL.  The
+ * previous token of row t is ids[t - 1] (chunk != 0, t > 0) or last_ids[slot_of[t]]; with `keep` last_ids takes in the newest
+ * tokens afterwards.  Tables bf16, turns [width / 2] double, everything on the device. */
+int blok_token_embedding(const uint32_t *ids, uint32_t *last_ids, const int *slot_of, const int *pos, int chunk, int keep,
+                         const blok_bf16_t *embed, int vocab, const blok_bf16_t *bigram, int buckets, long mul_prev,
+                         long mul_cur, float scale, const double *turns, int T, int width, int true_width, float *x,
+                         blok_stream_t stream);
+/* What a selective state space feeds its recurrence with.  proj Act (bf16, or fp32 with f32) [T, ld]: the convolution's
+ * inputs at column `first`, the step sizes at dt_at.
+ *   out    Act [T, channels]: silu(b + the causal convolution per channel); conv_w fp32 [taps, channels], current token last
+ *   ring   Act [slots, taps, channels]: a sequence's newest inputs, position p at p % taps; read and updated
+ *   token  fp32 [heads, token_ld, 4]: softplus(step + dt_bias), its product with rate[head] (the log decay), and that product's
+ *          running sum inside the token's 64-token chunk in two parts
+ * chunk != 0: T consecutive tokens of one sequence, else one token of each of T.  slot_of, pos int32 [T] in both cases. */
+int blok_state_inputs(const void *proj, int f32, int ld, int first, int dt_at, int heads, int channels, int taps,
+                      const float *conv_w, const float *conv_b, const float *dt_bias, const float *rate, void *ring,
+                      const int *slot_of, const int *pos, int T, int chunk, void *out, float *token, int token_ld,
+                      blok_stream_t stream);
+/* The recurrence: per head S = decay S + step B x^T, o = S^T C + skip x, S fp32 [slots, heads, state_dim, vdim].  xbc Act
+ * [T, ld]: x [heads * vdim] | B [groups * state_dim] | C [groups * state_dim]; `token` as above; the other arguments as in
+ * blok_linear_attention (scratch: blok_linear_attention_scratch_bytes(heads, state_dim, vdim, T)). */
+int blok_selective_state(const void *xbc, int f32, int ld, int heads, int groups, int state_dim, int vdim,
+                         const float *token, int token_ld, const float *skip, float *state, int slot, int first_pos, int T,
+                         const int *slot_of, const int *pos, float *o, void *scratch, blok_stream_t stream);
+/* out = v / rms(v) * w with v = o * silu(gate), the mean square over each of `parts` equal parts of the heads * true_vdim true
+ * columns.  Arguments as in blok_gated_norm. */
+int blok_gate_then_norm(const float *o, const void *gate, int ld_gate, const float *w, int heads, int vdim, int true_vdim,
+                        int parts, float eps, int T, void *out, int ld_out, int f32, blok_stream_t stream);
+
+/* Grouped softmax attention over a paged cache whose rows are [keys of every key head | values of every key head]; query head
+ * h reads key head h / (heads / kv_heads).  score = (q . k) * scale + bias[h][distance], softmax over positions 0..pos[i],
+ * head h's output times sigmoid(gate[i][h]).
+ *   bias   fp32 [heads, bias_len], its last entry for every distance from there on; NULL: none
+ *   gate   Act [T, ld_gate] or NULL; q Act [T, ldq] and out Act [T, ldo], head by head
+ * dim is a multiple of 32, vdim of 16.  blok_grouped_append: q | k | v rows (Act [T, ld]); q is normed in place by its root mean
+ * square over all heads (true_dim values each) times q_norm, k likewise, and the rows appended to the pool (pool NULL: only q;
+ * q_norm NULL: no norms). */
+int blok_grouped_append(void *qkv, int f32, int ld, int heads, int kv_heads, int dim, int true_dim, int vdim,
+                        const float *q_norm, const float *k_norm, float eps, const int *table, int table_stride,
+                        int page_rows, const int *slot_of, const int *pos, int T, void *pool, blok_stream_t stream);
+/* Entry i attends for the sequence in slot_of[i].  The workspace must be zero before the first call and serve calls of one T
+ * and max_ctx only. */
+size_t blok_grouped_attend_workspace_bytes(int heads, int kv_heads, int dim, int vdim, int T, long max_ctx);
+int blok_grouped_attend(const void *q, int f32, int ldq, const void *gate, int ld_gate, const void *pool, const int *table,
+                        int table_stride, int page_rows, const int *slot_of, const int *pos, int heads, int kv_heads,
+                        int dim, int vdim, float scale, const float *bias, int bias_len, int T, long max_ctx, void *out,
+                        int ldo, void *workspace, blok_stream_t stream);
+/* T queries of the sequence in `slot` at positions n - T .. n - 1 (bf16, tcgen05).  dim <= 256, vdim <= 128; without a bias the
+ * scale is positive.  page_rows is a multiple of 32; every row of the pool holds finite values. */
+int blok_grouped_prompt(const blok_bf16_t *q, int ldq, const blok_bf16_t *gate, int ld_gate, const blok_bf16_t *pool,
+                        long pool_rows, const int *table, int table_stride, int page_rows, int slot, int heads,
+                        int kv_heads, int dim, int vdim, float scale, const float *bias, int bias_len, int T, int n,
+                        blok_bf16_t *out, int ldo, blok_stream_t stream);
+/* out[t, r] = silu(w[r] . x[t]) * (w[R + r] . x[t]) on tcgen05: w bf16 [2 R, K], out bf16 [T, R]. */
+int blok_gemm_swiglu(const blok_bf16_t *x, const blok_bf16_t *w, int T, int R, int K, blok_bf16_t *out, blok_stream_t stream);
 /* out[t, r] = act(sum_k x[t, k] w[r, k]) on tcgen05 with TMA-fed tiles; act: none, or the square of ReLU. */
 int blok_gemm_bf16(const blok_bf16_t *x, const blok_bf16_t *w, int T, int R, int K, int relu2, blok_bf16_t *out_bf16,
                    float *out_f32, blok_stream_t stream);
@@ -583,6 +644,9 @@ int blok_model_destroy(blok_model_t *model);
  * picks one.  blok_model_architectures: their names, separated by spaces.
  *   Nomozen: a decoder of retention, lightning and latent-attention layers with table-routed squared-ReLU experts,
  *            Dynamic-Tanh norms and hyper-connected residual streams (csrc/nomozen.cu).
+ *   Pamopel: a decoder of selective state-space (Mamba-2) and grouped-attention layers (biases by distance, a gate per head,
+ *            keys and values that a layer borrows from an earlier one), SiLU-gated feed-forward, layer norms on both sides
+ *            of every sublayer, bigram and sinusoidal embeddings (csrc/pamopel.cu).
  * Such a model is always paged; slots, steps, prompts, generation and batching are the calls below, as for every model. */
 enum { BLOK_DTYPE_BF16 = 0, /* products and activations in bf16, fp32 accumulation; norms, scores, decays, recurrent states,
                                positions and the residual in fp32 */

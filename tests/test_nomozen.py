@@ -106,7 +106,7 @@ def test_configuration_errors_name_the_place(lib, tmp_path):
             else:
                 cfg[path[-1]] = value
         return setter
-    for path, value, message in ((("architecture",), "Unheard", "not one of: Nomozen"),
+    for path, value, message in ((("architecture",), "Unheard", 'architecture "Unheard" is not one of: '),
                                  (("layers", 0, "type"), "convolution", 'layer 0: unknown type "convolution"'),
                                  (("layers", 0, "mixer", "decay"), [0.5], "layer 0.mixer: decay has not one entry per head"),
                                  (("layers", 1, "mixer", "heads"), 0, "layer 1.mixer: heads is not a positive integer"),
