@@ -261,20 +261,23 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LaArgs a) {
   float4 *p = reinterpret_cast<float4 *>(a.chunk_state + (size_t)h * n + i);
   for (int c0 = 0; c0 < a.chunks; c0 += kAhead) {
     float4 own[kAhead];
-#pragma unroll
-    for (int j = 0; j < kAhead; ++j)
-      if (c0 + j < a.chunks) own[j] = p[(size_t)(c0 + j) * stride];
+    float decay[kAhead];
 #pragma unroll
     for (int j = 0; j < kAhead; ++j)
       if (c0 + j < a.chunks) {
         const int n = min(kLinChunk, a.T - (c0 + j) * kLinChunk);
-        float d;
         if (TOKEN) {
           const float4 w = a.token[(size_t)h * a.token_ld + (c0 + j) * kLinChunk + n - 1];
-          d = expf(w.z + w.w);
+          decay[j] = w.z + w.w;
         } else {
-          d = a.decay_pow[h * (kLinChunk + 1) + n];
+          decay[j] = a.decay_pow[h * (kLinChunk + 1) + n];
         }
+        own[j] = p[(size_t)(c0 + j) * stride];
+      }
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j)
+      if (c0 + j < a.chunks) {
+        const float d = TOKEN ? expf(decay[j]) : decay[j];
         p[(size_t)(c0 + j) * stride] = s;
         s = make_float4(fmaf(d, s.x, own[j].x), fmaf(d, s.y, own[j].y), fmaf(d, s.z, own[j].z), fmaf(d, s.w, own[j].w));
       }

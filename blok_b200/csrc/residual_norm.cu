@@ -7,11 +7,10 @@
 
 namespace blok {
 
-// The CTA's sum; s_red has one word per warp, and may be used again at once.
+// The CTA's sum; s_red has one word per warp and serves one call.
 template <int WARPS>
 __device__ __forceinline__ float rn_sum(float v, float *s_red) {
   v = warp_sum(v);
-  __syncthreads();
   if ((threadIdx.x & 31) == 0) s_red[threadIdx.x >> 5] = v;
   __syncthreads();
   v = s_red[0];
@@ -23,7 +22,7 @@ __device__ __forceinline__ float rn_sum(float v, float *s_red) {
 // v <- (v - mean) / sqrt(variance + eps) over the row's true columns (the thread's are 4 (tid + THREADS k) + j); columns of
 // the padding become 0.
 template <int THREADS, int KEEP>
-__device__ __forceinline__ void rn_layer_norm(float4 (&v)[KEEP], int width, float eps, float *s_red) {
+__device__ __forceinline__ void rn_layer_norm(float4 (&v)[KEEP], int width, float eps, float (*s_red)[THREADS / 32]) {
   auto each = [&](auto f) {
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
@@ -33,13 +32,13 @@ __device__ __forceinline__ void rn_layer_norm(float4 (&v)[KEEP], int width, floa
   };
   float s = 0.f;
   each([&](bool in, float &x) { s += in ? x : 0.f; });
-  const float mean = rn_sum<THREADS / 32>(s, s_red) / (float)width;
+  const float mean = rn_sum<THREADS / 32>(s, s_red[0]) / (float)width;
   s = 0.f;
   each([&](bool in, float &x) {
     x = in ? x - mean : 0.f;
     s = fmaf(x, x, s);
   });
-  const float r = 1.0f / sqrtf(rn_sum<THREADS / 32>(s, s_red) / (float)width + eps);
+  const float r = 1.0f / sqrtf(rn_sum<THREADS / 32>(s, s_red[1]) / (float)width + eps);
   each([&](bool, float &x) { x *= r; });
 }
 
@@ -50,10 +49,17 @@ __device__ __forceinline__ float4 rn_bf16x4(const uint16_t *p) {
 
 template <int THREADS, int KEEP>
 __global__ void __launch_bounds__(THREADS) residual_norm_kernel(const ResidualNorm a) {
-  __shared__ float s_red[THREADS / 32];
+  __shared__ float s_red[4][THREADS / 32];
   const int t = blockIdx.x, tid = threadIdx.x;
   float *xr = a.x + (size_t)t * a.width;
-  float4 x[KEEP];
+  float4 x[KEEP], w[KEEP];
+  if (a.norm_w) {  // on their way before the reductions
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int c = 4 * (tid + THREADS * k);
+      if (c < a.width) w[k] = *reinterpret_cast<const float4 *>(a.norm_w + c);
+    }
+  }
   if (a.ids) {
     const uint32_t last = (uint32_t)a.vocab - 1, id = min(a.ids[t], last);
     const int pos = a.pos ? a.pos[t] : 0;
@@ -98,20 +104,20 @@ __global__ void __launch_bounds__(THREADS) residual_norm_kernel(const ResidualNo
       if (c < a.width) x[k] = *reinterpret_cast<const float4 *>(xr + c);
     }
     if (a.y) {
-      float4 y[KEEP];
+      float4 y[KEEP], p[KEEP];
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         const int c = 4 * (tid + THREADS * k);
         y[k] = c < a.width ? *reinterpret_cast<const float4 *>(a.y + (size_t)t * a.width + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        p[k] = a.post_w && c < a.width ? *reinterpret_cast<const float4 *>(a.post_w + c) : make_float4(1.f, 1.f, 1.f, 1.f);
       }
       if (a.post_w) rn_layer_norm<THREADS, KEEP>(y, a.true_width, a.eps, s_red);
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         const int c = 4 * (tid + THREADS * k);
         if (c >= a.width) continue;
-        const float4 w = a.post_w ? *reinterpret_cast<const float4 *>(a.post_w + c) : make_float4(1.f, 1.f, 1.f, 1.f);
-        x[k] = make_float4(fmaf(a.mult, y[k].x * w.x, x[k].x), fmaf(a.mult, y[k].y * w.y, x[k].y), fmaf(a.mult, y[k].z * w.z, x[k].z),
-                           fmaf(a.mult, y[k].w * w.w, x[k].w));
+        x[k] = make_float4(fmaf(a.mult, y[k].x * p[k].x, x[k].x), fmaf(a.mult, y[k].y * p[k].y, x[k].y), fmaf(a.mult, y[k].z * p[k].z, x[k].z),
+                           fmaf(a.mult, y[k].w * p[k].w, x[k].w));
         *reinterpret_cast<float4 *>(xr + c) = x[k];
       }
     }
@@ -127,13 +133,12 @@ __global__ void __launch_bounds__(THREADS) residual_norm_kernel(const ResidualNo
     }
   }
   if (a.norm_w) {
-    rn_layer_norm<THREADS, KEEP>(x, a.true_width, a.eps, s_red);
+    rn_layer_norm<THREADS, KEEP>(x, a.true_width, a.eps, s_red + 2);
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
       const int c = 4 * (tid + THREADS * k);
       if (c >= a.width) continue;
-      const float4 w = *reinterpret_cast<const float4 *>(a.norm_w + c);
-      const float4 h = make_float4(x[k].x * w.x, x[k].y * w.y, x[k].z * w.z, x[k].w * w.w);
+      const float4 h = make_float4(x[k].x * w[k].x, x[k].y * w[k].y, x[k].z * w[k].z, x[k].w * w[k].w);
       const size_t at = (size_t)t * a.width + c;
       if (a.h_f32) *reinterpret_cast<float4 *>(static_cast<float *>(a.h) + at) = h;
       else *reinterpret_cast<uint2 *>(static_cast<uint16_t *>(a.h) + at) = make_uint2(pack_bf16x2(h.x, h.y), pack_bf16x2(h.z, h.w));
@@ -149,7 +154,7 @@ int launch_residual_norm(const ResidualNorm &a, cudaStream_t stream) {
   if (a.width <= 512) residual_norm_kernel<128, 1><<<a.T, 128, 0, stream>>>(a);
   else if (a.width <= 1024) residual_norm_kernel<256, 1><<<a.T, 256, 0, stream>>>(a);
   else if (a.width <= 2048) residual_norm_kernel<256, 2><<<a.T, 256, 0, stream>>>(a);
-  else if (a.width <= 4096) residual_norm_kernel<256, 4><<<a.T, 256, 0, stream>>>(a);
+  else if (a.width <= 4096) residual_norm_kernel<512, 2><<<a.T, 512, 0, stream>>>(a);
   else if (a.width <= 8192) residual_norm_kernel<512, 4><<<a.T, 512, 0, stream>>>(a);
   else residual_norm_kernel<1024, 8><<<a.T, 1024, 0, stream>>>(a);
   return launch_status("residual_norm_kernel");

@@ -1,37 +1,34 @@
 // What a selective state space (Mamba-2) feeds its recurrence with, and what follows it: the causal convolution per channel
 // with SiLU, step sizes and decays, and the gate with a norm over parts.  The recurrence itself is linear_attn.cu.
 //
-// A sequence's last inputs of the convolution live in a ring of `taps` rows, position p at p % taps: a token reads taps - 1
-// rows that it does not write, so a decode step reads and writes the ring in one launch.  A prompt reads the ring for its
-// first tokens and writes it in the launch after that.
+// A sequence's last inputs of the convolution live in a ring of `taps` rows, position p at p % taps.  Every channel of a ring is
+// read and written by one thread: the one that has the sequence's first tokens of the call, taps - 1 of them at least.
 #include "common.cuh"
 #include "stack_kernels.h"
 
 namespace blok {
 
-constexpr int kSiThreads = 256, kSiTokens = 8;  // tokens per thread of the convolution
+constexpr int kSiThreads = 256, kSiTokens = 4;  // tokens per thread of a long prompt's convolution
 
+// Eight channels of a row, as they are stored.
 template <typename Act>
-struct Si8 {  // eight channels
-  float v[8];
-  __device__ __forceinline__ void load(const Act *p) {
-    if constexpr (sizeof(Act) == 2) {
-      const uint4 u = *reinterpret_cast<const uint4 *>(p);
-      const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+struct Si8 {
+  static constexpr int kWords = sizeof(Act) * 2;
+  uint32_t w[kWords];
+  __device__ __forceinline__ void clear() {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) v[2 * j] = bf16lo(w[j]), v[2 * j + 1] = bf16hi(w[j]);
-    } else {
-      const float4 a = *reinterpret_cast<const float4 *>(p), b = *reinterpret_cast<const float4 *>(p + 4);
-      v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+    for (int i = 0; i < kWords; ++i) w[i] = 0;
+  }
+  __device__ __forceinline__ void load(const Act *p) {
+#pragma unroll
+    for (int i = 0; i < kWords; i += 4) {
+      const uint4 u = *reinterpret_cast<const uint4 *>(reinterpret_cast<const uint32_t *>(p) + i);
+      w[i] = u.x, w[i + 1] = u.y, w[i + 2] = u.z, w[i + 3] = u.w;
     }
   }
-  __device__ __forceinline__ void store(Act *p) const {
-    if constexpr (sizeof(Act) == 2) {
-      *reinterpret_cast<uint4 *>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
-    } else {
-      *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
-      *reinterpret_cast<float4 *>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
-    }
+  __device__ __forceinline__ float value(int i) const {
+    if constexpr (sizeof(Act) == 2) return i & 1 ? bf16hi(w[i / 2]) : bf16lo(w[i / 2]);
+    else return __uint_as_float(w[i]);
   }
 };
 template <typename Act>
@@ -40,51 +37,86 @@ __device__ __forceinline__ void si_copy8(Act *dst, const Act *src) {
   if constexpr (sizeof(Act) == 4) *reinterpret_cast<uint4 *>(dst + 4) = *reinterpret_cast<const uint4 *>(src + 4);
 }
 
-// Channels [c, c + 8) of tokens t0 .. t0 + n - 1.
-template <typename Act>
+// Channels [c, c + 8) of tokens t0 .. t0 + n - 1, n <= TOKENS.  TAPS: a.taps if it is known (every load is on its way before the
+// first use then), or 0.
+template <typename Act, int TAPS, int TOKENS>
 __device__ __forceinline__ void si_conv(const StateInputs &a, const StackRows &r, int c, int t0, int n, bool chunk) {
   const Act *x = static_cast<const Act *>(a.proj) + a.first + c;
-  Act *ring = static_cast<Act *>(a.ring) + c;
-  Si8<Act> bias;
+  const Act *ring = static_cast<const Act *>(a.ring) + c;
+  // the input of token t0 + q, q possibly negative: of this call, of the ring (a step's tokens have rings of their own), or zeros
+  auto input = [&](int t, int back, Si8<Act> *in) {
+    if (back == 0 || (chunk && t >= back)) {
+      in->load(x + (size_t)(t - back) * a.ld);
+      return;
+    }
+    const int p = r.pos[t] - back;
+    if (p >= 0) in->load(ring + ((size_t)r.slot_of[t] * a.taps + p % a.taps) * a.channels);
+    else in->clear();
+  };
+  Si8<float> bias;
+  bias.load(a.conv_b + c);
+  float acc[TOKENS][8];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) bias.v[i] = a.conv_b[c + i];
-  Si8<Act> acc[kSiTokens];
+  for (int q = 0; q < TOKENS; ++q)
 #pragma unroll
-  for (int q = 0; q < kSiTokens; ++q) acc[q] = bias;
-  for (int j = a.taps - 1; j >= 0; --j) {  // the input j tokens back
-    float w[8];
-    const float4 w0 = *reinterpret_cast<const float4 *>(a.conv_w + (size_t)(a.taps - 1 - j) * a.channels + c),
-                 w1 = *reinterpret_cast<const float4 *>(a.conv_w + (size_t)(a.taps - 1 - j) * a.channels + c + 4);
-    w[0] = w0.x, w[1] = w0.y, w[2] = w0.z, w[3] = w0.w, w[4] = w1.x, w[5] = w1.y, w[6] = w1.z, w[7] = w1.w;
+    for (int i = 0; i < 8; ++i) acc[q][i] = bias.value(i);
+  auto add = [&](const Si8<float> &w, const Si8<Act> &in, float (&to)[8]) {
 #pragma unroll
-    for (int q = 0; q < kSiTokens; ++q) {
-      const int t = t0 + q;
-      if (q >= n) break;
-      Si8<Act> in;
-      if (j == 0 || (chunk && t >= j)) {
-        in.load(x + (size_t)(t - j) * a.ld);
-      } else {
-        const int p = r.pos[t] - j;
-        if (p < 0) continue;  // zeros before the start
-        in.load(ring + ((size_t)r.slot_of[t] * a.taps + p % a.taps) * a.channels);
+    for (int i = 0; i < 8; ++i) to[i] = fmaf(w.value(i), in.value(i), to[i]);
+  };
+  if constexpr (TAPS > 0) {
+    Si8<float> w[TAPS];
+    Si8<Act> in[TOKENS + TAPS - 1];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j].load(a.conv_w + (size_t)j * a.channels + c);
+#pragma unroll
+    for (int k = 0; k < TOKENS + TAPS - 1; ++k) {
+      const int q = k - (TAPS - 1);  // token t0 + q, seen from token t0 if it lies in front of it
+      if (q < n) input(q < 0 ? t0 : t0 + q, q < 0 ? -q : 0, &in[k]);
+    }
+#pragma unroll
+    for (int q = 0; q < TOKENS; ++q)
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+        if (q < n) add(w[j], in[q + j], acc[q]);
+  } else {
+    for (int j = 0; j < a.taps; ++j) {
+      Si8<float> w;
+      w.load(a.conv_w + (size_t)j * a.channels + c);
+#pragma unroll
+      for (int q = 0; q < TOKENS; ++q) {
+        if (q >= n) break;
+        Si8<Act> in;
+        input(t0 + q, a.taps - 1 - j, &in);
+        add(w, in, acc[q]);
       }
-#pragma unroll
-      for (int i = 0; i < 8; ++i) acc[q].v[i] = fmaf(w[i], in.v[i], acc[q].v[i]);
     }
   }
 #pragma unroll
-  for (int q = 0; q < kSiTokens; ++q) {
+  for (int q = 0; q < TOKENS; ++q) {
     if (q >= n) break;
+    float v[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const float z = acc[q].v[i];
-      acc[q].v[i] = sizeof(Act) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : z / (1.0f + expf(-z));  // bf16: rounded right away
+      const float z = acc[q][i];
+      v[i] = sizeof(Act) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : z / (1.0f + expf(-z));  // bf16: rounded right away
     }
-    acc[q].store(static_cast<Act *>(a.out) + (size_t)(t0 + q) * a.channels + c);
+    Act *out = static_cast<Act *>(a.out) + (size_t)(t0 + q) * a.channels + c;
+    if constexpr (sizeof(Act) == 2) {
+      *reinterpret_cast<uint4 *>(out) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+    } else {
+      *reinterpret_cast<float4 *>(out) = make_float4(v[0], v[1], v[2], v[3]);
+      *reinterpret_cast<float4 *>(out + 4) = make_float4(v[4], v[5], v[6], v[7]);
+    }
   }
-  if (!chunk)
-    for (int q = 0; q < n; ++q)
-      si_copy8(ring + ((size_t)r.slot_of[t0 + q] * a.taps + r.pos[t0 + q] % a.taps) * a.channels, x + (size_t)(t0 + q) * a.ld);
+}
+
+// The newest inputs of a call go into the ring: rows t0 .. t0 + n - 1.
+template <typename Act>
+__device__ __forceinline__ void si_keep(const StateInputs &a, const StackRows &r, int c, int t0, int n) {
+  for (int t = t0; t < t0 + n; ++t)
+    si_copy8(static_cast<Act *>(a.ring) + ((size_t)r.slot_of[t] * a.taps + r.pos[t] % a.taps) * a.channels + c,
+             static_cast<const Act *>(a.proj) + (size_t)t * a.ld + a.first + c);
 }
 
 // 32 heads (one per lane), the 64 tokens of chunk `chunk_index` (eight per warp): step, log decay, running sum.
@@ -123,57 +155,52 @@ __device__ __forceinline__ void si_steps(const StateInputs &a, int head0, int ch
   }
 }
 
-// Blocks 0 .. conv_blocks - 1: convolution; then `ring_blocks` that write the ring; then the steps.
-template <typename Act>
-__global__ void __launch_bounds__(kSiThreads) state_inputs_kernel(const StateInputs a, const StackRows r, int T, int chunk, int per_thread,
-                                                                  int conv_blocks, int ring_blocks) {
-  const int per = a.channels / 8;
-  int b = blockIdx.x;
-  if (b < conv_blocks) {
-    const long u = (long)b * kSiThreads + threadIdx.x;
-    const int c = (int)(u % per) * 8, t0 = (int)(u / per) * per_thread;
-    if (t0 < T) si_conv<Act>(a, r, c, t0, min(per_thread, T - t0), chunk != 0);
+// The steps in the first `step_blocks` blocks, then the convolution: unit 0 of a chunk has its first `lead` tokens.
+template <typename Act, int TAPS, int TOKENS>
+__global__ void __launch_bounds__(kSiThreads, sizeof(Act) == 2 ? 2 : 1) state_inputs_kernel(const StateInputs a, const StackRows r, int T, int chunk, int lead, int step_blocks) {
+  const int b = (int)blockIdx.x - step_blocks;
+  if (b < 0) {
+    const int groups = (a.heads + 31) / 32;
+    si_steps<Act>(a, (int)blockIdx.x % groups * 32, (int)blockIdx.x / groups, T);
     return;
   }
-  b -= conv_blocks;
-  if (b < ring_blocks) {  // the last `taps` inputs of a prompt's portion
+  const int per = a.channels / 8, u = b * kSiThreads + (int)threadIdx.x, i = u / per, c = (u - i * per) * 8;
+  if (!chunk) {
+    if (i >= T) return;
+    si_conv<Act, TAPS, 1>(a, r, c, i, 1, false);
+    si_keep<Act>(a, r, c, i, 1);
+    return;
+  }
+  int t0 = i == 0 ? 0 : lead + (i - 1) * TOKENS;
+  const int end = min(T, i == 0 ? lead : t0 + TOKENS);
+  for (; t0 < end; t0 += TOKENS) si_conv<Act, TAPS, TOKENS>(a, r, c, t0, min(TOKENS, end - t0), true);
+  if (i == 0) {
     const int n = min(T, a.taps);
-    const long u = (long)b * kSiThreads + threadIdx.x;
-    const int c = (int)(u % per) * 8, i = (int)(u / per);
-    if (i < n) {
-      const int t = T - n + i;
-      si_copy8(static_cast<Act *>(a.ring) + ((size_t)r.slot_of[t] * a.taps + r.pos[t] % a.taps) * a.channels + c,
-               static_cast<const Act *>(a.proj) + (size_t)t * a.ld + a.first + c);
-    }
-    return;
+    si_keep<Act>(a, r, c, T - n, n);
   }
-  b -= ring_blocks;
-  const int groups = (a.heads + 31) / 32;
-  si_steps<Act>(a, b % groups * 32, b / groups, T);
 }
 
-template <typename Act>
+template <typename Act, int TAPS, int TOKENS>
 static int state_inputs(const StateInputs &a, const StackRows &r, int T, bool chunk, cudaStream_t stream) {
-  const long per = a.channels / 8;
-  // several tokens per thread where that leaves enough threads: neighbours share most inputs
-  const int per_thread = chunk && per * T >= (long)kSiTokens * sm_count() * kSiThreads ? kSiTokens : chunk && per * T >= 2l * sm_count() * kSiThreads ? 2 : 1;
-  const auto blocks = [&](long units) { return (int)((units + kSiThreads - 1) / kSiThreads); };
-  const int conv = blocks(per * ((T + per_thread - 1) / per_thread)), ring = blocks(per * (T < a.taps ? T : a.taps));
+  const int lead = chunk && a.taps > 1 ? a.taps - 1 : 1;
+  const long units = chunk ? 1 + (T > lead ? (T - lead + TOKENS - 1) / TOKENS : 0) : T, threads = a.channels / 8 * units;
   const int steps = (a.heads + 31) / 32 * ((T + kLinChunk - 1) / kLinChunk);
-  if (!chunk) {
-    state_inputs_kernel<Act><<<conv + steps, kSiThreads, 0, stream>>>(a, r, T, 0, per_thread, conv, 0);
-    return launch_status("state_inputs_kernel");
-  }
-  state_inputs_kernel<Act><<<conv, kSiThreads, 0, stream>>>(a, r, T, 1, per_thread, conv, 0);
-  if (int rc = launch_status("state_inputs_kernel")) return rc;
-  state_inputs_kernel<Act><<<ring + steps, kSiThreads, 0, stream>>>(a, r, T, 1, 1, 0, ring);
+  BLOK_REQUIRE(threads < (1l << 30), BLOK_ERR_SHAPE, "state space: %d channels of %d tokens", a.channels, T);
+  state_inputs_kernel<Act, TAPS, TOKENS><<<steps + (int)((threads + kSiThreads - 1) / kSiThreads), kSiThreads, 0, stream>>>(a, r, T, chunk, lead, steps);
   return launch_status("state_inputs_kernel");
+}
+template <typename Act>
+static int state_inputs_of(const StateInputs &a, const StackRows &r, int T, bool chunk, cudaStream_t stream) {
+  // several tokens per thread where that leaves enough threads: neighbours share most inputs
+  const bool many = (long)a.channels / 8 * T / kSiTokens >= 512l * sm_count();
+  if (a.taps != 4) return many ? state_inputs<Act, 0, kSiTokens>(a, r, T, chunk, stream) : state_inputs<Act, 0, 1>(a, r, T, chunk, stream);
+  return many ? state_inputs<Act, 4, kSiTokens>(a, r, T, chunk, stream) : state_inputs<Act, 4, 1>(a, r, T, chunk, stream);
 }
 
 int launch_state_inputs(const StateInputs &a, const StackRows &r, int T, bool chunk, cudaStream_t stream) {
   BLOK_REQUIRE(a.heads >= 1 && a.channels % 16 == 0 && a.taps >= 1 && a.ld % 8 == 0 && a.first % 8 == 0 && T >= 1 && T <= a.token_ld, BLOK_ERR_SHAPE,
                "state space: %d heads, %d channels, %d taps", a.heads, a.channels, a.taps);
-  return a.f32 ? state_inputs<float>(a, r, T, chunk, stream) : state_inputs<uint16_t>(a, r, T, chunk, stream);
+  return a.f32 ? state_inputs_of<float>(a, r, T, chunk, stream) : state_inputs_of<uint16_t>(a, r, T, chunk, stream);
 }
 
 // ---- gate, then a norm over equal parts of the true columns.  grid = (T, parts) ----
