@@ -22,7 +22,7 @@ constexpr int kGtKStep = 64;
 
 template <int BN>
 struct GtCfg {
-  static constexpr int kStages = BN == 128 ? 3 : 4;
+  static constexpr int kStages = BN == 128 ? 3 : 2;  // 96 KB: two CTAs per SM, one computes while the other stores
   static constexpr int kABytes = kGtTileRows * 128, kBBytes = BN * 128;
   static constexpr int kStageBytes = kABytes + kBBytes;
   static constexpr int kSmem = kStages * kStageBytes + 1024;  // + 1,024: the slices start on a 1,024-byte boundary
@@ -107,22 +107,26 @@ __global__ void __launch_bounds__(kGtThreads)
       for (int c = max(0, issued - S); c < issued; ++c) tp_wait(full + 8 * (c % S), (uint32_t)((c / S) & 1));
     }
   } else if (warp == 5) {
-    if (lane == 0) {
-      for (int c = 0; c < nsteps; ++c) {
-        const int s = c % S;
-        if (!tp_wait(full + 8 * s, (uint32_t)((c / S) & 1))) {
-          failed = true;
-          break;
-        }
-        tc_fence_after();
-        const uint64_t ad = tp_desc_k_sw128(sbase + (uint32_t)s * Cfg::kStageBytes);
-        const uint64_t bd = tp_desc_k_sw128(sbase + (uint32_t)s * Cfg::kStageBytes + Cfg::kABytes);
+    // the whole warp walks the slices, so that addresses and descriptors stay warp-uniform; one lane issues
+    const bool issues = tp_elect();
+    int s = 0;
+    uint32_t turn = 0;
+    for (int c = 0; c < nsteps; ++c) {
+      if (!__all_sync(0xffffffffu, tp_wait(full + 8 * s, turn))) {
+        failed = true;
+        break;
+      }
+      tc_fence_after();
+      const uint64_t ad = tp_desc_k_sw128(sbase + (uint32_t)s * Cfg::kStageBytes);
+      const uint64_t bd = tp_desc_k_sw128(sbase + (uint32_t)s * Cfg::kStageBytes + Cfg::kABytes);
+      if (issues) {
 #pragma unroll
         for (int k = 0; k < kGtKStep / 16; ++k)
           tp_mma(tmem, ad + (uint64_t)(2 * k), bd + (uint64_t)(2 * k), tp_idesc_bf16(BN), (c | k) ? 1u : 0u);
         tp_commit(empty + 8 * s);
+        if (c == nsteps - 1) tp_commit(done);
       }
-      if (!failed) tp_commit(done);
+      if (++s == S) s = 0, turn ^= 1;
     }
   } else {
     failed = !tp_wait(done, 0);

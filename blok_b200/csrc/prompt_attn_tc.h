@@ -24,10 +24,11 @@ struct PromptAttn {
   int bias_len = 0;
   const int *table = nullptr;   // pages of the sequence, `page_rows` rows each (a multiple of `box`); NULL: key j is row j
   int page_rows = 1, box = 64;  // box: rows per copied box of the key maps, 64 or 32
+  int stages = 0;               // tiles of 64 keys in shared memory at a time (set by the launch)
 };
 bool prompt_attn_supports(int dim, int vdim);
 // Maps of 64 columns, bf16, 128-byte swizzle (gemm_operand_map): boxes of 128 queries, of `box` keys.
-int launch_prompt_attn(const CUtensorMap &mq, const CUtensorMap &mkv, const CUtensorMap &mkr, const PromptAttn &a, cudaStream_t stream);
+int launch_prompt_attn(const CUtensorMap &mq, const CUtensorMap &mkv, const CUtensorMap &mkr, PromptAttn a, cudaStream_t stream);
 int prompt_attn_take_error(unsigned *out);
 
 }  // namespace blok

@@ -38,6 +38,18 @@ __device__ __forceinline__ bool tp_wait(uint32_t mbar, uint32_t parity) {
   }
   return false;
 }
+// True in one lane of a converged warp.
+__device__ __forceinline__ bool tp_elect() {
+  uint32_t is;
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p;\n\t"
+      "elect.sync _|p, 0xffffffff;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t"
+      "}\n"
+      : "=r"(is));
+  return is != 0;
+}
 // One box of a 2-D tensor map (x: column in elements, 16-byte aligned; y: row) into shared memory, counted on the mbarrier.
 __device__ __forceinline__ void tp_load_2d(uint32_t dst, const CUtensorMap *map, int x, int y, uint32_t mbar) {
   asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
