@@ -1,7 +1,7 @@
 """The streaming kernels keep compiling for sm_100a within their register and spill limits (nvcc cross-compiles
 without a GPU).  Fused decode kernel: 512 threads per CTA leave 128 registers per thread, and the two streaming loops,
 where the kernel spends its time, must not spill at all.  Small-group kernel, weight-streaming bf16 kernel, the
-tcgen05 GEMMs, the prompt attention and the chunked linear attention: the registers their CTAs per SM allow, and next to nothing on the stack."""
+tcgen05 GEMMs, the prompt and grouped attention and the chunked linear attention: the registers their CTAs per SM allow, and next to nothing on the stack."""
 import os
 import shutil
 import subprocess
@@ -49,11 +49,12 @@ def test_fused_kernel_registers_and_spills(tmp_path):
     ("wgemm_stream.cu", "wgemm_stream_kernel", 128, 16),
     # 288 threads, two CTAs per SM (tensor memory and shared memory are sized for two): 113 registers at most
     ("wgemm_tc.cu", "wgemm_tc_kernel", 112, 16),
-    # 192 threads: the softmax rows of the prompt kernel live in registers; two GEMM CTAs per SM at the 128-row tile
-    ("prompt_attn_tc.cu", "prompt_attn_tc_kernel", 255, 0),
+    # 320 threads: half a softmax row per thread lives in registers; two GEMM CTAs per SM
+    ("prompt_attn_tc.cu", "prompt_attn_tc_kernel", 128, 0),
     ("gemm_tma.cu", "gemm_tma_kernel", 80, 0),
-    # 256 threads, two CTAs per SM
+    # 256 threads, two CTAs per SM (one where a CTA has 32 query heads or values over 128)
     ("linear_attn.cu", "linear_chunk_out_kernel", 128, 0),
+    ("grouped_attn.cu", "grouped_attend_kernel", 160, 0),
 ])
 def test_streaming_kernels_registers_and_spills(tmp_path, source, kernel, max_regs, max_spill):
     out = str(tmp_path / (source + ".cubin"))
