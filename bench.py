@@ -364,7 +364,7 @@ def pamopel_config(width, heads, q_heads, kv_heads, ff, vocab=32768):
     state = {"heads": heads, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
     attn = {"heads": q_heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "bias_max": 128}
     return {"architecture": "Pamopel", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "logit_scale": 1.0,
-            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 1009, "mul_cur": 17}},
             "layers": [{"type": "mamba2", "mixer": state, "mlp": mlp}, {"type": "attention", "mixer": attn, "mlp": mlp},
                        {"type": "attention", "mixer": dict(attn, kv_from=1), "mlp": mlp}, {"type": "mamba2", "mixer": state, "mlp": mlp}]}
 

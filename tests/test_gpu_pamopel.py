@@ -340,7 +340,7 @@ def grouped_inputs(rng, n, H, G, d, dv, pos):
 
 
 @pytest.mark.parametrize("H,G,d,dv,blen,dtype", [
-    (1, 1, 32, 16, 1, torch.bfloat16), (6, 2, 64, 80, 65, torch.bfloat16), (16, 1, 96, 96, 240, torch.bfloat16), (32, 8, 128, 128, 0, torch.bfloat16),
+    (1, 1, 32, 16, 1, torch.bfloat16), (6, 2, 64, 80, 65, torch.bfloat16), (14, 1, 96, 112, 210, torch.bfloat16), (32, 8, 128, 128, 0, torch.bfloat16),
     (40, 2, 64, 64, 129, torch.bfloat16), (3, 3, 160, 208, 500, torch.bfloat16), (17, 1, 256, 256, 33, torch.bfloat16), (4, 2, 320, 272, 40, torch.bfloat16),
     (6, 3, 96, 48, 70, torch.float32), (5, 1, 32, 16, 0, torch.float32)])
 @pytest.mark.parametrize("page", [32, 64])
@@ -363,7 +363,7 @@ def test_grouped_attend(cuda, H, G, d, dv, blen, dtype, page):
         assert np.max(np.abs(got[i] - want[i])) < bar * np.abs(want[i]).max(), p
 
 
-@pytest.mark.parametrize("H,G,d,dv,blen", [(1, 1, 32, 16, 1), (6, 2, 64, 80, 65), (8, 1, 96, 96, 240), (4, 2, 128, 128, 0), (3, 3, 160, 64, 500),
+@pytest.mark.parametrize("H,G,d,dv,blen", [(1, 1, 32, 16, 1), (6, 2, 64, 80, 65), (10, 2, 96, 112, 210), (4, 2, 128, 128, 0), (3, 3, 160, 64, 500),
                                            (2, 1, 256, 112, 33), (5, 5, 224, 48, 1000)])
 @pytest.mark.parametrize("T,n,page", [(33, 33, 32), (200, 200, 64), (64, 321, 32), (129, 257, 96), (40, 1000, 64)])
 def test_grouped_prompt(cuda, H, G, d, dv, blen, T, n, page):
